@@ -1,3 +1,3 @@
 """Importing this package registers every architecture the engine ships."""
 
-from . import bumalix, gekopel, goganex, llama, nerenex, zomolix  # noqa: F401
+from . import bumalix, dogotar, gekopel, goganex, llama, nerenex, zomolix  # noqa: F401

@@ -214,6 +214,41 @@ PRESETS.update({
 })
 
 
+def _dogotar(width: int, vocab: int, groups: int, heads: int, kv_heads: int, ff: int, window: int) -> dict:
+    """``groups`` times (attention, parallel, parallel), every layer with a feed-forward."""
+    mlp = {"kind": "dense", "ff": ff}
+    attention = {"type": "attention", "mlp": mlp,
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                           "mask": {"size": window}, "v_mix": True, "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0}}}}
+    parallel = {"type": "parallel", "mlp": mlp,
+                "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                                   "mask": {"size": window}}, "left_scale": 0.5,
+                          "right": {"heads": heads // 2, "dim": 128, "vdim": 128, "gate_cap": 15.0}, "right_scale": 0.5}}
+    return {"architecture": "Dogotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": [attention, parallel, parallel] * groups}
+
+
+PRESETS.update({
+    "dogotar-tiny": {
+        "architecture": "Dogotar", "vocab": 256, "width": 64, "norm": {"eps": 1e-6},
+        "layers": [
+            {"type": "attention", "mlp": {"kind": "dense", "ff": 128},
+             "mixer": {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "softcap": 30.0, "mask": {"size": 24}, "v_mix": True,
+                       "rot": {"base": 10000.0, "dims": 8, "scaling": {"factor": 4.0}}}},
+            {"type": "parallel", "mlp": None,
+             "mixer": {"left": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 32, "scale": 0.25, "softcap": 20.0, "mask": {"size": 40}},
+                       "left_scale": 0.7, "right": {"heads": 3, "dim": 16, "vdim": 24, "gate_cap": 10.0}, "right_scale": 0.6}},
+            {"type": "attention", "mlp": {"kind": "dense", "ff": 96},
+             "mixer": {"heads": 2, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "softcap": 30.0, "mask": {"size": 16}, "v_mix": True,
+                       "rot": {"base": 10000.0, "dims": 16}}},
+        ],
+    },
+    # layer sizes of a 1B- and an 8B-class decoder (width, heads, feed-forward), for the benchmarks: heads and windows of
+    # Bumalix's presets
+    "dogotar-2048": _dogotar(2048, 32768, 4, 16, 4, 8192, 1024),
+    "dogotar-4096": _dogotar(4096, 32768, 3, 32, 8, 14336, 2048),
+})
+
+
 def preset(name: str):
     """The typed configuration of a preset, read by its architecture's own reader."""
     try:

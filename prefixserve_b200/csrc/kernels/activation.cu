@@ -1,4 +1,5 @@
-// Activations of a feed-forward without a gate branch, out = act(x) element by element, float32 arithmetic:
+// Activations of a feed-forward without a gate branch, out = act(x) element by element, float32 arithmetic (rows of the result
+// may be runs of columns of wider ones):
 //   silu, gelu_tanh (as in the gated kernels), and xielu with two learned numbers (p, q):
 //     z > 0:  softplus(p) z^2 + z/2
 //     z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2
@@ -18,7 +19,7 @@ __device__ __forceinline__ float softplusf_(float x) { return log1pf(expf(-fabsf
 
 template <typename T>
 __global__ void unary_act_kernel(const T* __restrict__ x, T* __restrict__ out, size_t total, int code,
-                                 const float* __restrict__ params) {
+                                 const float* __restrict__ params, size_t cols, size_t ldo) {
   pdl_trigger();
   pdl_wait();
   float ap = 0.f, aq = 0.f;
@@ -32,13 +33,13 @@ __global__ void unary_act_kernel(const T* __restrict__ x, T* __restrict__ out, s
     if (code == UNARY_XIELU) v = z > 0.f ? ap * z * z + 0.5f * z : aq * (expm1f(z) - z) + 0.5f * z;
     else if (code == UNARY_RELU2) v = relu2f_(z);
     else v = gate_act(z, code);
-    out[i] = from_float<T>(v);
+    out[cols == ldo ? i : i / cols * ldo + i % cols] = from_float<T>(v);
   }
 }
 
 // Eight bfloat16 elements a thread (16-byte loads and stores).
 __global__ void unary_act_vec_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ out, size_t vecs, int code,
-                                     const float* __restrict__ params) {
+                                     const float* __restrict__ params, size_t cols8, size_t ldo8) {
   pdl_trigger();
   pdl_wait();
   float ap = 0.f, aq = 0.f;
@@ -67,7 +68,7 @@ __global__ void unary_act_vec_kernel(const __nv_bfloat16* __restrict__ x, __nv_b
       }
       o2[k] = __floats2bfloat162_rn(a, b);
     }
-    reinterpret_cast<uint4*>(out)[i] = o4;
+    reinterpret_cast<uint4*>(out)[cols8 == ldo8 ? i : i / cols8 * ldo8 + i % cols8] = o4;
   }
 }
 
@@ -210,23 +211,25 @@ PSB_API int psb_gate_mul(const void* x, int x_dtype, const void* gate, void* out
   return 0;
 }
 
-PSB_API int psb_unary_act(const void* x, int dtype, void* out, long long total, int code, const void* params,
-                          cudaStream_t stream) {
+// (x [total / cols, cols], dtype, out in rows ldo numbers apart, total, cols, ldo, code, params or null, stream)
+PSB_API int psb_unary_act(const void* x, int dtype, void* out, long long total, long long cols, long long ldo, int code,
+                          const void* params, cudaStream_t stream) {
+  if (cols < 1 || ldo < cols || total % cols) PSB_REFUSE("unary_act: %lld numbers in rows of %lld, %lld apart", total, cols, ldo);
   if (total < 0) PSB_REFUSE("unary_act: negative size");
   if (code < 0 || code > UNARY_RELU2) PSB_REFUSE("unary_act: activation code %d is not built", code);
   if (code == UNARY_XIELU && !params) PSB_REFUSE("unary_act: xielu needs its two numbers");
   if (total == 0) return 0;
-  if (dtype == PSB_BF16 && total % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
+  if (dtype == PSB_BF16 && cols % 8 == 0 && ldo % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
     const long long vecs = total / 8, vblocks = (vecs + 255) / 256;
     psb_launch(unary_act_vec_kernel, dim3((unsigned)(vblocks > 148 * 16 ? 148 * 16 : vblocks)), dim3(256), 0, stream,
-               (const __nv_bfloat16*)x, (__nv_bfloat16*)out, (size_t)vecs, code, (const float*)params);
+               (const __nv_bfloat16*)x, (__nv_bfloat16*)out, (size_t)vecs, code, (const float*)params, (size_t)(cols / 8), (size_t)(ldo / 8));
     PSB_LAUNCH_CHECK("unary_act");
     return 0;
   }
   const long long blocks = (total + 255) / 256;
   PSB_DISPATCH_DTYPE(dtype, T, {
     psb_launch(unary_act_kernel<T>, dim3((unsigned)(blocks > 65535 * 16 ? 65535 * 16 : blocks)), dim3(256), 0, stream,
-               (const T*)x, (T*)out, (size_t)total, code, (const float*)params);
+               (const T*)x, (T*)out, (size_t)total, code, (const float*)params, (size_t)cols, (size_t)ldo);
   });
   PSB_LAUNCH_CHECK("unary_act");
   return 0;

@@ -1,11 +1,15 @@
 // Causal grouped-query attention over the paged cache for designs whose scores carry more than q.k:
 //
-//   score(i, j) = (q_i . k_j) * scale + bias[h][min(i - j, reach - 1)]       (bias optional)
+//   score(i, j) = cap((q_i . k_j) * scale) + bias[h][min(i - j, reach - 1)]  (bias optional; cap(s) = softcap * tanh(s / softcap),
+//             optional)
 //   visible:  j <= i,  j > i - window (window optional),  floor(j / chunk) == floor(i / chunk) (chunk optional);
 //             with ``keep_first`` > 0 (and a window, no chunk) the first keep_first keys of the sequence stay visible
 //             to every later query, at their true positions: j <= i and (j > i - window or j < keep_first)
 //   weights = exp(score) / (sum over visible j of exp(score) + exp(sink[h]))  (sink optional: a term of the
 //             denominator that has no key and no value)
+//
+//   out = (sum of weights * values) * out_scale * sigmoid(gate)              (gate optional, a number per token, head and value
+//             channel; rows of ``out`` and of ``gate`` may be runs of columns of wider ones)
 //
 // Keys and values may have different sizes (dim, vdim); the cache entry holds one row per token and key/value head,
 // [num_pages, 1, hkv, page_size, dim + vdim]: the key, then the value.  ``bias`` is a float32 table
@@ -31,6 +35,19 @@ namespace {
 
 constexpr int WARPS = 4;
 constexpr int MAX_D = 256;
+
+// The cap on the scores and what is done to a finished row on its way out.
+struct RowsTail {
+  const void* gate;  // pre-activations of an output gate, rows ldg numbers apart, or null
+  long long ldg, ldo;
+  float out_scale, softcap;  // softcap 0: none
+};
+
+template <typename T>
+__device__ __forceinline__ float tail_factor(const RowsTail& tail, size_t t, int column) {
+  if (!tail.gate) return tail.out_scale;
+  return tail.out_scale / (1.f + expf(-to_float<T>(static_cast<const T*>(tail.gate)[t * tail.ldg + column])));
+}
 
 template <typename T, typename TKV>
 __global__ void attention_biased_append_kernel(const T* __restrict__ qkv, const int32_t* __restrict__ positions,
@@ -109,7 +126,7 @@ attention_biased_kernel(const T* __restrict__ q, const TKV* __restrict__ kv, con
                         const float* __restrict__ bias, const float* __restrict__ sink, T* __restrict__ out, int T_tokens,
                         int hq, int hkv, int dim, int vdim, int page_size, int window, int chunk, int reach, float scale,
                         const int32_t* __restrict__ item_start, int skip_from, int keep_first, float* __restrict__ partial,
-                        int splits) {
+                        int splits, const RowsTail tail) {
   __shared__ __align__(16) float qs[MAX_D];
   __shared__ float part[WARPS][MAX_D + 2];
   pdl_trigger();
@@ -161,6 +178,7 @@ attention_biased_kernel(const T* __restrict__ q, const TKV* __restrict__ kv, con
       const int page = pages[key / page_size];
       off = (long long)((size_t)page * page_elems + (size_t)g * head_stride + (size_t)(key % page_size) * rw);
       s = dot_row<TKV>(qs, kv + off, dim, vec) * scale;
+      if (tail.softcap > 0.f) s = tail.softcap * tanhf(s / tail.softcap);
       if (brow) s += brow[min(p - key, reach - 1)];
     }
     const float m_new = fmaxf(m, warp_max(s));
@@ -230,11 +248,11 @@ attention_biased_kernel(const T* __restrict__ q, const TKV* __restrict__ kv, con
     return;
   }
   const float inv = 1.f / L;
-  T* orow = out + ((size_t)t * hq + h) * vdim;
+  T* orow = out + (size_t)t * tail.ldo + (size_t)h * vdim;
 #pragma unroll
   for (int i = 0; i < MAX_D / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < vdim) orow[d] = from_float<T>(acc[i] * inv);
+    if (d < vdim) orow[d] = from_float<T>(acc[i] * inv * tail_factor<T>(tail, t, h * vdim + d));
   }
 }
 
@@ -244,7 +262,7 @@ constexpr int MAX_KEY_SPLITS = 16;
 template <typename T>
 __global__ void __launch_bounds__(32)
 attention_biased_merge_kernel(const float* __restrict__ partial, const float* __restrict__ sink, T* __restrict__ out, int hq,
-                              int vdim, int splits) {
+                              int vdim, int splits, const RowsTail tail) {
   pdl_trigger();
   pdl_wait();
   const size_t unit = blockIdx.x;  // token * hq + head
@@ -279,11 +297,12 @@ attention_biased_merge_kernel(const float* __restrict__ partial, const float* __
     }
   }
   const float inv = 1.f / L;
-  T* orow = out + unit * vdim;
+  const size_t t = unit / hq;
+  T* orow = out + t * tail.ldo + (size_t)h * vdim;
 #pragma unroll
   for (int i = 0; i < MAX_D / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < vdim) orow[d] = from_float<T>(acc[i] * inv);
+    if (d < vdim) orow[d] = from_float<T>(acc[i] * inv * tail_factor<T>(tail, t, h * vdim + d));
   }
 }
 
@@ -300,7 +319,7 @@ attention_biased_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
                              const int32_t* __restrict__ table, int table_width, const int32_t* __restrict__ positions,
                              const int32_t* __restrict__ item_start, int items, int min_tokens, const float* __restrict__ bias,
                              const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int hq, int hkv, int dim, int vdim,
-                             int page_size, int window, int chunk, int reach, float scale, int keep_first) {
+                             int page_size, int window, int chunk, int reach, float scale, int keep_first, const RowsTail tail) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -391,6 +410,7 @@ attention_biased_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
         float dot = 0.f;
         for (int d = 0; d < dim; ++d) dot = fmaf(qq[d], ks[d * 33 + lane], dot);
         s = dot * scale;
+        if (tail.softcap > 0.f) s = tail.softcap * tanhf(s / tail.softcap);
         if (bias) s += bias[(size_t)hh * reach + min(p - key, reach - 1)];
       }
       float m = st[2 * u], l = st[2 * u + 1];
@@ -420,7 +440,8 @@ attention_biased_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     const int u = i / VP, d = i - u * VP;
     if (d >= vdim) continue;
     const int tt = u / share, hh = g * share + (u - tt * share);
-    out[((size_t)(t0 + tt) * hq + hh) * vdim + d] = __float2bfloat16_rn(accs[i] / st[2 * u + 1]);
+    out[(size_t)(t0 + tt) * tail.ldo + (size_t)hh * vdim + d] =
+        __float2bfloat16_rn(accs[i] / st[2 * u + 1] * tail_factor<__nv_bfloat16>(tail, t0 + tt, hh * vdim + d));
   }
 }
 
@@ -454,7 +475,7 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int32_t* __restrict__ table, int table_width, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ item_start, int items, int min_tokens, const float* __restrict__ bias,
                             const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int hq, int hkv, int dim, int vdim,
-                            int page_size, int window, int chunk, int reach, float scale, int keep_first) {
+                            int page_size, int window, int chunk, int reach, float scale, int keep_first, const RowsTail tail) {
   constexpr int KS = D + 8, VS = MMA_KEYS + 8;  // row pitches that keep the fragment loads off each other's banks
   __shared__ __align__(16) __nv_bfloat16 ks[MMA_KEYS * KS];   // keys [key][d]; first the tile's queries [row][d]
   __shared__ __align__(16) __nv_bfloat16 vt[V * VS];          // values transposed [v][key]
@@ -577,6 +598,15 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       }
     }
     float top[2] = {-FLT_MAX, -FLT_MAX};
+    if (tail.softcap > 0.f) {
+      // cap * tanh(s * scale / cap) / scale as cap / scale * (1 - 2 / (exp(2 s scale / cap) + 1)): an error of a few units in
+      // the last place of the cap, far out it reaches +-cap (the scale itself is applied below)
+      const float far = tail.softcap / scale, rate = 2.f * PSB_LOG2E / far;
+#pragma unroll
+      for (int n = 0; n < MMA_KEYS / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[n][e] = fmaf(-2.f * far, __fdividef(1.f, exp2f(sc[n][e] * rate) + 1.f), far);
+    }
 #pragma unroll
     for (int n = 0; n < MMA_KEYS / 8; ++n) {
 #pragma unroll
@@ -647,11 +677,13 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const int row = warp * 16 + gid + 8 * r;
     if (row >= nt) continue;
     const float inv = 1.f / l[r];
-    __nv_bfloat16* orow = out + ((size_t)(t0 + row) * hq + h) * vdim;
+    __nv_bfloat16* orow = out + (size_t)(t0 + row) * tail.ldo + (size_t)h * vdim;
 #pragma unroll
     for (int nv = 0; nv < V / 8; ++nv) {
       const int c = nv * 8 + 2 * tig;
-      if (c < vdim) *reinterpret_cast<uint32_t*>(orow + c) = pack_bf16(o[nv][2 * r] * inv, o[nv][2 * r + 1] * inv);
+      if (c < vdim)
+        *reinterpret_cast<uint32_t*>(orow + c) = pack_bf16(o[nv][2 * r] * (inv * tail_factor<__nv_bfloat16>(tail, t0 + row, h * vdim + c)),
+                                                           o[nv][2 * r + 1] * (inv * tail_factor<__nv_bfloat16>(tail, t0 + row, h * vdim + c + 1)));
     }
   }
 }
@@ -688,12 +720,15 @@ PSB_API int psb_attention_biased_append(const void* qkv, int dtype, const void* 
 
 // ``skip_from`` > 0: tokens of portions with at least that many tokens are left to the tiled kernel (item_start needed).
 // (q, dtype, kv, kv_dtype, table, table_width, positions, token_item, bias, sink, out, T, hq, hkv, dim, vdim, page_size,
-//  window, chunk, reach, scale, item_start, skip_from, keep_first, partial [T * hq, splits, vdim + 2] float32 or null, splits, stream)
+//  window, chunk, reach, scale, item_start, skip_from, keep_first, partial [T * hq, splits, vdim + 2] float32 or null, splits,
+//  gate, ldg, ldo, out_scale, softcap, stream); gate (or null) has the type of q
 PSB_API int psb_attention_biased(const void* q, int dtype, const void* kv, int kv_dtype, const void* table, int table_width,
                                  const void* positions, const void* token_item, const void* bias, const void* sink, void* out,
                                  int T, int hq, int hkv, int dim, int vdim, int page_size, int window, int chunk, int reach,
                                  float scale, const void* item_start, int skip_from, int keep_first, void* partial, int splits,
-                                 cudaStream_t stream) {
+                                 const void* gate, long long ldg, long long ldo, float out_scale, float softcap, cudaStream_t stream) {
+  if (ldo < (long long)hq * vdim || (gate && ldg < (long long)hq * vdim) || softcap < 0.f) PSB_REFUSE("attention_biased: bad output or gate rows, or a negative cap");
+  const RowsTail tail{gate, ldg, ldo, out_scale, softcap};
   if (splits < 1 || splits > MAX_KEY_SPLITS || (splits > 1 && (!partial || skip_from > 0)))
     PSB_REFUSE("attention_biased: 1 to %d shares of the keys (with their scratch, and no tokens left to another kernel), not %d", MAX_KEY_SPLITS, splits);
   if (keep_first < 0 || (keep_first > 0 && (window < 1 || chunk > 0))) PSB_REFUSE("attention_biased: kept first keys go with a window and no chunk mask");
@@ -710,14 +745,14 @@ PSB_API int psb_attention_biased(const void* q, int dtype, const void* kv, int k
       psb_launch(attention_biased_kernel<T_, TKV>, dim3((unsigned)blocks, (unsigned)splits), dim3(WARPS * 32), 0, stream, (const T_*)q,
                  (const TKV*)kv, (const int32_t*)table, table_width, (const int32_t*)positions, (const int32_t*)token_item,
                  (const float*)bias, (const float*)sink, (T_*)out, T, hq, hkv, dim, vdim, page_size, window, chunk, reach, scale,
-                 (const int32_t*)item_start, skip_from, keep_first, (float*)partial, splits);
+                 (const int32_t*)item_start, skip_from, keep_first, (float*)partial, splits, tail);
     });
   });
   PSB_LAUNCH_CHECK("attention_biased");
   if (splits > 1) {
     PSB_DISPATCH_DTYPE(dtype, T_, {
       psb_launch(attention_biased_merge_kernel<T_>, dim3((unsigned)blocks), dim3(32), 0, stream, (const float*)partial,
-                 (const float*)sink, (T_*)out, hq, vdim, splits);
+                 (const float*)sink, (T_*)out, hq, vdim, splits, tail);
     });
     PSB_LAUNCH_CHECK("attention_biased_merge");
   }
@@ -732,11 +767,16 @@ PSB_API int psb_attention_biased_mma_supported(int hq, int hkv, int dim, int vdi
 // The tensor-core kernel over every portion of at least ``min_tokens`` tokens (bfloat16; grid sized by an upper bound on
 // the 64-token tiles).  Other tokens are left untouched.
 // (q, kv, table, table_width, positions, item_start, items, T, min_tokens, bias, sink, out, hq, hkv, dim, vdim,
-//  page_size, window, chunk, reach, scale, keep_first, stream)
+//  page_size, window, chunk, reach, scale, keep_first, gate, ldg, ldo, out_scale, softcap, stream)
 PSB_API int psb_attention_biased_mma(const void* q, const void* kv, const void* table, int table_width, const void* positions,
                                      const void* item_start, int items, int T, int min_tokens, const void* bias, const void* sink,
                                      void* out, int hq, int hkv, int dim, int vdim, int page_size, int window, int chunk, int reach,
-                                     float scale, int keep_first, cudaStream_t stream) {
+                                     float scale, int keep_first, const void* gate, long long ldg, long long ldo, float out_scale,
+                                     float softcap, cudaStream_t stream) {
+  if (ldo < (long long)hq * vdim || ldo % 2 || ((uintptr_t)out & 3) || (gate && ldg < (long long)hq * vdim) || softcap < 0.f)
+    PSB_REFUSE("attention_biased_mma: bad output or gate rows, or a negative cap");
+  if (softcap > 0.f && scale == 0.f) PSB_REFUSE("attention_biased_mma: a cap needs a scale that is not zero");
+  const RowsTail tail{gate, ldg, ldo, out_scale, softcap};
   if (!psb_attention_biased_mma_supported(hq, hkv, dim, vdim)) PSB_REFUSE("attention_biased_mma: shape not taken");
   if (keep_first < 0 || (keep_first > 0 && (window < 1 || chunk > 0))) PSB_REFUSE("attention_biased_mma: kept first keys go with a window and no chunk mask");
   if (page_size < 1 || table_width < 1 || window < 0 || chunk < 0 || (bias && reach < 1)) PSB_REFUSE("attention_biased_mma: bad arguments");
@@ -747,7 +787,7 @@ PSB_API int psb_attention_biased_mma(const void* q, const void* kv, const void* 
   psb_launch(attention_biased_mma_kernel<D_, V_>, grid, block, 0, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv,    \
              (const int32_t*)table, table_width, (const int32_t*)positions, (const int32_t*)item_start, items, min_tokens,     \
              (const float*)bias, (const float*)sink, (__nv_bfloat16*)out, hq, hkv, dim, vdim, page_size, window, chunk, reach, \
-             scale, keep_first)
+             scale, keep_first, tail)
   if (dim <= 64 && vdim <= 64) MMA_CASE(64, 64);
   else if (dim <= 64) MMA_CASE(64, 128);
   else if (vdim <= 64) MMA_CASE(128, 64);
@@ -770,12 +810,15 @@ PSB_API int psb_attention_biased_tile_supported(int hq, int hkv, int dim, int vd
 // The tiled kernel over every portion of at least ``min_tokens`` tokens (the grid is sized by an upper bound on their
 // tiles, so its shape depends on T and the number of items only).  Other tokens are left untouched.
 // (q, kv, table, table_width, positions, item_start, items, T, min_tokens, bias, sink, out, hq, hkv, dim, vdim,
-//  page_size, window, chunk, reach, scale, keep_first, stream)
+//  page_size, window, chunk, reach, scale, keep_first, gate, ldg, ldo, out_scale, softcap, stream)
 PSB_API int psb_attention_biased_tiles(const void* q, const void* kv, const void* table, int table_width, const void* positions,
                                        const void* item_start, int items, int T, int min_tokens,
                                        const void* bias, const void* sink, void* out, int hq, int hkv, int dim, int vdim,
                                        int page_size, int window, int chunk, int reach, float scale, int keep_first,
+                                       const void* gate, long long ldg, long long ldo, float out_scale, float softcap,
                                        cudaStream_t stream) {
+  if (ldo < (long long)hq * vdim || (gate && ldg < (long long)hq * vdim) || softcap < 0.f) PSB_REFUSE("attention_biased_tiles: bad output or gate rows, or a negative cap");
+  const RowsTail tail{gate, ldg, ldo, out_scale, softcap};
   if (keep_first < 0 || (keep_first > 0 && (window < 1 || chunk > 0))) PSB_REFUSE("attention_biased_tiles: kept first keys go with a window and no chunk mask");
   if (items < 1 || T < 1 || min_tokens < 1) return 0;
   const int tiles = (T + TILE_T - 1) / TILE_T + items;
@@ -797,7 +840,7 @@ PSB_API int psb_attention_biased_tiles(const void* q, const void* kv, const void
     psb_launch(kernel, grid, block, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv, (const int32_t*)table,    \
                table_width, (const int32_t*)positions, (const int32_t*)item_start, items, min_tokens,                          \
                (const float*)bias, (const float*)sink, (__nv_bfloat16*)out, hq, hkv, dim, vdim,                                \
-               page_size, window, chunk, reach, scale, keep_first);                                                            \
+               page_size, window, chunk, reach, scale, keep_first, tail);                                                      \
     launched = true;                                                                                                           \
   }
 #define TILE_ROW(DP_) TILE_CASE(DP_, 32) TILE_CASE(DP_, 64) TILE_CASE(DP_, 128) TILE_CASE(DP_, 256)

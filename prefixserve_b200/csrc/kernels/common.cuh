@@ -115,6 +115,13 @@ __device__ __forceinline__ float gate_act(float g, int act) {
   return g / (1.f + expf(-g));
 }
 
+// The same functions where the result is rounded to bfloat16 anyway (epilogues of the tensor-core products): the tanh form of
+// GELU as z * sigmoid(2u), u = sqrt(2/pi) (z + 0.044715 z^3), since (1 + tanh u) / 2 = sigmoid(2u).
+__device__ __forceinline__ float quick_act(float z, int act) {
+  const float e = act == PSB_ACT_GELU_TANH ? 1.5957691216057308f * z * fmaf(0.044715f * z, z, 1.f) : z;
+  return __fdividef(z, 1.f + __expf(-e));
+}
+
 // A gated feed-forward whose two branches are clipped before they meet: g = min(gate, limit), u = clamp(up, -limit, limit),
 // value = g * sigmoid(alpha * g) * (u + offset).  It has numbers of its own, so it is no PsbAct code that every entry
 // point takes: kernels that know it receive PSB_ACT_CLIPPED together with a GluClip.

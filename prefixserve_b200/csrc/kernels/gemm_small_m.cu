@@ -210,7 +210,7 @@ gemm_stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
         const float up = __bfloat162float(__float2bfloat16_rn(v[TILES - 1]));
         out = gated_value(gate, up, act, clip);
       } else {
-        out = v[0];
+        out = act < 0 ? v[0] : gate_act(v[0], act);  // act -1: the sums as they are
       }
       y[(size_t)m * ldy + row] = from_float<TOut>(out);
     }
@@ -243,11 +243,24 @@ PSB_API int psb_gemm_stream(const void* x, const void* W, void* y, int out_dtype
   if (M < 0 || M > 16 || N < 1 || K < 32 || K % 32 || sms < 1) PSB_REFUSE("gemm_stream: needs M <= 16 and K a multiple of 32 (M=%d N=%d K=%d)", M, N, K);
   if (M == 0) return 0;
   int rc;
-  if (out_dtype == PSB_F32) rc = M <= 8 ? launch_stream<1, 1, float>(x, W, y, M, N, K, N, 0, 0, sms, stream) : launch_stream<2, 1, float>(x, W, y, M, N, K, N, 0, 0, sms, stream);
-  else if (out_dtype == PSB_BF16) rc = M <= 8 ? launch_stream<1, 1, __nv_bfloat16>(x, W, y, M, N, K, N, 0, 0, sms, stream) : launch_stream<2, 1, __nv_bfloat16>(x, W, y, M, N, K, N, 0, 0, sms, stream);
+  if (out_dtype == PSB_F32) rc = M <= 8 ? launch_stream<1, 1, float>(x, W, y, M, N, K, N, 0, -1, sms, stream) : launch_stream<2, 1, float>(x, W, y, M, N, K, N, 0, -1, sms, stream);
+  else if (out_dtype == PSB_BF16) rc = M <= 8 ? launch_stream<1, 1, __nv_bfloat16>(x, W, y, M, N, K, N, 0, -1, sms, stream) : launch_stream<2, 1, __nv_bfloat16>(x, W, y, M, N, K, N, 0, -1, sms, stream);
   else PSB_REFUSE("gemm_stream: unknown output dtype %d", out_dtype);
   if (rc) return rc;
   PSB_LAUNCH_CHECK("gemm_stream");
+  return 0;
+}
+
+// y[M,N] = f(x W^T) in bfloat16, f the activation named by its code (PsbAct), in rows ldy numbers apart.
+PSB_API int psb_gemm_stream_unary(const void* x, const void* W, void* y, int M, int N, int K, int ldy, int sms, int activation,
+                                  cudaStream_t stream) {
+  if (!psb_activation_known(activation)) PSB_REFUSE("gemm_stream_unary: activation code %d is not built", activation);
+  if (M < 0 || M > 16 || N < 1 || K < 32 || K % 32 || sms < 1 || ldy < N) PSB_REFUSE("gemm_stream_unary: needs M <= 16, K a multiple of 32 and rows that hold N (M=%d N=%d K=%d ldy=%d)", M, N, K, ldy);
+  if (M == 0) return 0;
+  const int rc = M <= 8 ? launch_stream<1, 1, __nv_bfloat16>(x, W, y, M, N, K, ldy, 0, activation, sms, stream)
+                        : launch_stream<2, 1, __nv_bfloat16>(x, W, y, M, N, K, ldy, 0, activation, sms, stream);
+  if (rc) return rc;
+  PSB_LAUNCH_CHECK("gemm_stream_unary");
   return 0;
 }
 

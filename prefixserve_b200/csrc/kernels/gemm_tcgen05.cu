@@ -68,13 +68,15 @@ using namespace tc;
 // mode: 0 plain (C[M, N], tile columns [n0, n0+BN/2) and [n0+BN/2, n0+BN)); 1 gated (C[M, I], W = [gate; up], tile
 // columns [n0, n0+128) of the gate and the same of the up rows); 2 the projection of an attention layer (columns as in
 // 0; the epilogue rotates queries and keys and stores queries, keys and values where RopeArgs says, C is not used).
-enum : int { MODE_PLAIN = 0, MODE_GATED = 1, MODE_ROPE = 2, MODE_GATED_GELU = 3, MODE_RELU2 = 4, MODE_GATED_CLIPPED = 5, MODE_GATED_SCALED = 6 };
+enum : int { MODE_PLAIN = 0, MODE_GATED = 1, MODE_ROPE = 2, MODE_GATED_GELU = 3, MODE_RELU2 = 4, MODE_GATED_CLIPPED = 5, MODE_GATED_SCALED = 6,
+             MODE_SILU = 7, MODE_GELU = 8 };
 // gated: SiLU, the tanh form of GELU, or (clipped) g * sigmoid(alpha g) * (u + offset) with g = min(gate, limit) and
 // u = clamp(up, -limit, limit), the three numbers in a GluClip (common.cuh).
 using GluArgs = GluClip;
 __device__ __forceinline__ bool mode_is_gated(int mode) { return mode == MODE_GATED || mode == MODE_GATED_GELU || mode == MODE_GATED_CLIPPED || mode == MODE_GATED_SCALED; }
 __device__ __forceinline__ float clipped_gate(float g, float u, const GluArgs& a) { return clipped_gate_value(g, u, a); }
-// MODE_RELU2: columns as in 0, the epilogue stores max(sum, 0)^2.
+// MODE_RELU2: columns as in 0, the epilogue stores max(sum, 0)^2.  MODE_SILU, MODE_GELU: the same with SiLU or the tanh form of
+// GELU of the sum.
 //
 // Grouped products (``tile_expert`` given): W is a stack of matrices [experts * N_out, K] and every 128-row tile of A
 // belongs to one of them, named by tile_expert[row tile] (-1: the tile holds no rows and is skipped by all three
@@ -355,6 +357,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 if (mode == MODE_RELU2) {
                   v0 = fmaxf(v0, 0.f), v1 = fmaxf(v1, 0.f);
                   v0 *= v0, v1 *= v1;
+                } else if (mode == MODE_SILU || mode == MODE_GELU) {
+                  const int act = mode == MODE_SILU ? PSB_ACT_SILU : PSB_ACT_GELU_TANH;
+                  v0 = quick_act(v0, act), v1 = quick_act(v1, act);
                 }
                 packed[q] = pack2(v0, v1);
               }
@@ -423,8 +428,10 @@ int choose_width(int M, int N_out, bool gated, bool rope, int D, int sms) {
 
 int launch(const void* a, const void* w, void* c, int M, int w_rows, int N_out, int K, int up_offset, int mode, int sms,
            cudaStream_t stream, const RopeArgs& rope = RopeArgs{}, const int32_t* tile_expert = nullptr,
-           const GluArgs& glu = GluArgs{}, const float* row_scale = nullptr) {
+           const GluArgs& glu = GluArgs{}, const float* row_scale = nullptr, int ldc = 0) {
   const bool gated = mode == MODE_GATED || mode == MODE_GATED_GELU || mode == MODE_GATED_CLIPPED || mode == MODE_GATED_SCALED;
+  if (ldc == 0) ldc = N_out;
+  if (ldc < N_out) PSB_REFUSE("gemm_tcgen05: output rows %d numbers apart do not hold %d", ldc, N_out);
   if (M < 1 || N_out < 1 || K < 8 || K % 8) PSB_REFUSE("gemm_tcgen05: needs K a multiple of 8 (M=%d N=%d K=%d)", M, N_out, K);
   if (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c) & 15) PSB_REFUSE("gemm_tcgen05: operands must be 16-byte aligned");
   const int m_blocks = (M + BM - 1) / BM;
@@ -445,7 +452,7 @@ int launch(const void* a, const void* w, void* c, int M, int w_rows, int N_out, 
       configured.set();                                                                                              \
     }                                                                                                                \
     psb_launch(gemm_tcgen05_kernel<BN, HB>, dim3(grid), dim3(THREADS), (size_t)Tile<BN>::SMEM_BYTES, stream, map_a,   \
-               map_w, (__nv_bfloat16*)c, M, N_out, K, N_out, up_offset, mode, rope, tile_expert, glu, row_scale);    \
+               map_w, (__nv_bfloat16*)c, M, N_out, K, ldc, up_offset, mode, rope, tile_expert, glu, row_scale);      \
   } while (0)
   // the usual head sizes keep a row's angles in registers; every other multiple of 16 fetches them block by block
   if (mode == MODE_ROPE && rope.D == 128) { if (bn == 128) PSB_TCGEN05(128, 8); else PSB_TCGEN05(256, 8); }
@@ -464,6 +471,13 @@ int launch(const void* a, const void* w, void* c, int M, int w_rows, int N_out, 
 // C[M,N] = A[M,K] W[N,K]^T, all bfloat16 row-major, K % 8 == 0.  sms: CTAs to launch at most (the SM count).
 PSB_API int psb_gemm_tcgen05(const void* a, const void* w, void* c, int M, int N, int K, int sms, cudaStream_t stream) {
   return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, sms, stream);
+}
+
+// C[M,N] = f(A W^T), f the activation named by its code (PsbAct), in rows ldc numbers apart.
+PSB_API int psb_gemm_tcgen05_unary(const void* a, const void* w, void* c, int M, int N, int K, int ldc, int sms, int activation,
+                                   cudaStream_t stream) {
+  if (!psb_activation_known(activation)) PSB_REFUSE("gemm_tcgen05_unary: activation code %d is not built", activation);
+  return launch(a, w, c, M, N, N, K, 0, activation == PSB_ACT_SILU ? MODE_SILU : MODE_GELU, sms, stream, RopeArgs{}, nullptr, GluArgs{}, nullptr, ldc);
 }
 
 // act[M,I] = f(A Wg^T) * (A Wu^T) for W = [Wg; Wu] of shape [2I, K], f the activation named by its code (PsbAct).

@@ -51,6 +51,7 @@ struct Barriers {
 static_assert(sizeof(Barriers) <= 256, "room kept for the barriers");
 
 enum : int { MODE_PLAIN = 0, MODE_GATED = 1, MODE_ROPE = 2 };
+constexpr int NO_ACT = -1;  // plain products: the sums as they are, else the activation named by its code
 
 constexpr int SSQ_PITCH = 64;  // floats per tile in the array of partial sums of squares: one per row of A
 
@@ -308,6 +309,10 @@ gemm_fewrows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             ss = warp_sum(ss);  // a warp a token
             if ((e & 31) == 0) norm.ssq_out[tile * SSQ_PITCH + t] = ss;
           } else {
+            if (activation != NO_ACT) {
+#pragma unroll
+              for (int i = 0; i < 4; ++i) o[i] = gate_act(o[i], activation);
+            }
             store4(C + (size_t)t * ldc, col, N_out, aligned, o);
           }
           continue;
@@ -454,7 +459,7 @@ int choose_splits(int tiles, int k_blocks) {
 
 template <int MT>
 int launch_shape(const void* a, const void* w, void* c, int M, int w_rows, int N_out, int K, int up_offset, int mode, int activation,
-                 cudaStream_t stream, const RopeArgs& rope, const NormArgs& norm) {
+                 cudaStream_t stream, const RopeArgs& rope, const NormArgs& norm, int ldc) {
   static PsbPerDevice configured;  // more than 48 KB of dynamic shared memory has to be asked for once
   if (!configured.get()) {
     cudaError_t e = cudaFuncSetAttribute(gemm_fewrows_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<MT>::SMEM_BYTES);
@@ -468,7 +473,7 @@ int launch_shape(const void* a, const void* w, void* c, int M, int w_rows, int N
   const int tiles = (N_out + n_span - 1) / n_span;
   const int k_blocks = (K + BK - 1) / BK;
   const int ks = choose_splits<MT>(tiles, k_blocks);
-  cudaError_t e = launch_kernel<MT>(dim3(ks, tiles), stream, map_w, map_x, (__nv_bfloat16*)c, M, N_out, K, N_out, up_offset, mode,
+  cudaError_t e = launch_kernel<MT>(dim3(ks, tiles), stream, map_w, map_x, (__nv_bfloat16*)c, M, N_out, K, ldc, up_offset, mode,
                                     activation, rope, norm);
   if (e != cudaSuccess) {
     cudaGetLastError();
@@ -478,21 +483,29 @@ int launch_shape(const void* a, const void* w, void* c, int M, int w_rows, int N
 }
 
 int launch(const void* a, const void* w, void* c, int M, int w_rows, int N_out, int K, int up_offset, int mode, int activation,
-           cudaStream_t stream, const RopeArgs& rope = RopeArgs{}, const NormArgs& norm = NormArgs{}) {
+           cudaStream_t stream, const RopeArgs& rope = RopeArgs{}, const NormArgs& norm = NormArgs{}, int ldc = 0) {
+  if (ldc == 0) ldc = N_out;
+  if (ldc < N_out) PSB_REFUSE("gemm_fewrows: output rows %d numbers apart do not hold %d", ldc, N_out);
   if (norm.ssq_in && (norm.ssq_parts < 1 || !(norm.eps > 0.f))) PSB_REFUSE("gemm_fewrows: the norm in front needs its parts and a positive eps");
   if (norm.stream && (mode != MODE_PLAIN || !norm.gain || !norm.gained || !norm.ssq_out || (((uintptr_t)norm.stream | (uintptr_t)norm.gained) & 15)))
     PSB_REFUSE("gemm_fewrows: a product in front of a norm is a plain one with stream, gain, gained rows and shares given (16-byte aligned)");
   if (M < 1 || M > 64 || N_out < 1 || K < 8 || K % 8) PSB_REFUSE("gemm_fewrows: needs 1..64 rows and K a multiple of 8 (M=%d N=%d K=%d)", M, N_out, K);
   if (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c) & 15) PSB_REFUSE("gemm_fewrows: operands must be 16-byte aligned");
-  if (M <= 32) return launch_shape<32>(a, w, c, M, w_rows, N_out, K, up_offset, mode, activation, stream, rope, norm);
-  return launch_shape<64>(a, w, c, M, w_rows, N_out, K, up_offset, mode, activation, stream, rope, norm);
+  if (M <= 32) return launch_shape<32>(a, w, c, M, w_rows, N_out, K, up_offset, mode, activation, stream, rope, norm, ldc);
+  return launch_shape<64>(a, w, c, M, w_rows, N_out, K, up_offset, mode, activation, stream, rope, norm, ldc);
 }
 
 }  // namespace
 
 // C[M,N] = A[M,K] W[N,K]^T, all bfloat16 row-major, M <= 64, K % 8 == 0.
 PSB_API int psb_gemm_fewrows(const void* a, const void* w, void* c, int M, int N, int K, cudaStream_t stream) {
-  return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, 0, stream);
+  return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, NO_ACT, stream);
+}
+
+// C[M,N] = f(A W^T), f the activation named by its code (PsbAct), in rows ldc numbers apart.
+PSB_API int psb_gemm_fewrows_unary(const void* a, const void* w, void* c, int M, int N, int K, int ldc, int activation, cudaStream_t stream) {
+  if (!psb_activation_known(activation)) PSB_REFUSE("gemm_fewrows_unary: activation code %d is not built", activation);
+  return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, activation, stream, RopeArgs{}, NormArgs{}, ldc);
 }
 
 // act[M,I] = f(A Wg^T) * (A Wu^T) for W = [Wg; Wu] of shape [2I, K], f the activation named by its code (PsbAct).
@@ -533,7 +546,7 @@ NormArgs behind_norm(const void* ssq_in, int ssq_parts, float eps, int width) {
 // (ssq_in [ssq_parts][64] float32, from psb_gemm_fewrows_add_norm): every sum is scaled by rsqrt(sum(v^2) / K + eps).
 PSB_API int psb_gemm_fewrows_scaled(const void* a, const void* w, void* c, int M, int N, int K, const void* ssq_in, int ssq_parts,
                                     float eps, cudaStream_t stream) {
-  return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, 0, stream, RopeArgs{}, behind_norm(ssq_in, ssq_parts, eps, K));
+  return launch(a, w, c, M, N, N, K, 0, MODE_PLAIN, NO_ACT, stream, RopeArgs{}, behind_norm(ssq_in, ssq_parts, eps, K));
 }
 PSB_API int psb_gemm_fewrows_gated_scaled(const void* a, const void* w, void* act, int M, int I, int K, int activation,
                                           const void* ssq_in, int ssq_parts, float eps, cudaStream_t stream) {
@@ -566,7 +579,7 @@ PSB_API int psb_gemm_fewrows_add_norm(const void* a, const void* w, void* stream
                                       int M, int N, int K, cudaStream_t stream) {
   NormArgs n{};
   n.stream = (float*)stream_io; n.gain = (const float*)gain; n.gained = (__nv_bfloat16*)gained; n.ssq_out = (float*)ssq_out;
-  return launch(a, w, gained, M, N, N, K, 0, MODE_PLAIN, 0, stream, RopeArgs{}, n);
+  return launch(a, w, gained, M, N, N, K, 0, MODE_PLAIN, NO_ACT, stream, RopeArgs{}, n);
 }
 
 // For tests: 1, 2, 4 or 8 makes every later product cut the contraction into that many ranges (where it has that many

@@ -20,7 +20,7 @@
 // A portion of one chunk takes the last kernel alone, from and to the slot.
 //
 // normed_readout_kernel (a warp per token and head): o / sqrt(mean(o^2) + eps) * gain[vdim] * gate, rounded to the compute
-// type; the gate is read as it is or through silu.
+// type; the gate is read as it is, through silu or through a sigmoid; the gain is shared by the heads or each head has its own.
 #include "common.cuh"
 
 namespace {
@@ -300,12 +300,13 @@ linear_attention_starts_kernel(const float* __restrict__ state, long long slot_f
   }
 }
 
-enum : int { READOUT_GATE_PLAIN = 0, READOUT_GATE_SILU = 1 };
+enum : int { READOUT_GATE_PLAIN = 0, READOUT_GATE_SILU = 1, READOUT_GATE_SIGMOID = 2 };
 
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(128)
 normed_readout_kernel(const float* __restrict__ o, const TG* __restrict__ gate, long long ldg, int gate_act,
-                      const float* __restrict__ gain, TO* __restrict__ out, long long units, int H, int vdim, float eps) {
+                      const float* __restrict__ gain, int head_gains, TO* __restrict__ out, long long ldo, long long units, int H,
+                      int vdim, float eps) {
   pdl_trigger();
   pdl_wait();
   const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -318,10 +319,12 @@ normed_readout_kernel(const float* __restrict__ o, const TG* __restrict__ gate, 
   float ss = 0.f;
   for (int j = lane; j < vdim; j += 32) ss = fmaf(row[j], row[j], ss);
   const float inv = 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
-  TO* dst = out + (size_t)unit * vdim;
+  TO* dst = out + (size_t)t * ldo + (size_t)h * vdim;
+  if (head_gains) gain += (size_t)h * vdim;
   for (int j = lane; j < vdim; j += 32) {
     float v = to_float<TG>(g[j]);
     if (gate_act == READOUT_GATE_SILU) v = v / (1.f + expf(-v));
+    else if (gate_act == READOUT_GATE_SIGMOID) v = 1.f / (1.f + expf(-v));
     dst[j] = from_float<TO>(row[j] * inv * gain[j] * v);
   }
 }
@@ -386,17 +389,20 @@ PSB_API int psb_linear_attention(const void* proj, int dtype, long long ld, cons
   return 0;
 }
 
-// (o float32 [T, H, vdim], gate, gate_dtype, ldg, gate_act, gain, out, out_dtype, T, H, vdim, eps, stream)
-PSB_API int psb_normed_readout(const void* o, const void* gate, int gate_dtype, long long ldg, int gate_act, const void* gain, void* out,
-                               int out_dtype, int T, int H, int vdim, float eps, cudaStream_t stream) {
-  if (T < 0 || H < 1 || vdim < 1 || ldg < (long long)H * vdim) PSB_REFUSE("normed_readout: bad sizes H=%d vdim=%d ldg=%lld", H, vdim, ldg);
-  if (gate_act != READOUT_GATE_PLAIN && gate_act != READOUT_GATE_SILU) PSB_REFUSE("normed_readout: gate code %d is not built", gate_act);
+// (o float32 [T, H, vdim], gate, gate_dtype, ldg, gate_act, gain [vdim] or with head_gains [H, vdim], head_gains, out in rows ldo
+// numbers apart, out_dtype, ldo, T, H, vdim, eps, stream)
+PSB_API int psb_normed_readout(const void* o, const void* gate, int gate_dtype, long long ldg, int gate_act, const void* gain,
+                               int head_gains, void* out, int out_dtype, long long ldo, int T, int H, int vdim, float eps,
+                               cudaStream_t stream) {
+  if (T < 0 || H < 1 || vdim < 1 || ldg < (long long)H * vdim || ldo < (long long)H * vdim)
+    PSB_REFUSE("normed_readout: bad sizes H=%d vdim=%d ldg=%lld ldo=%lld", H, vdim, ldg, ldo);
+  if (gate_act != READOUT_GATE_PLAIN && gate_act != READOUT_GATE_SILU && gate_act != READOUT_GATE_SIGMOID) PSB_REFUSE("normed_readout: gate code %d is not built", gate_act);
   if (T == 0) return 0;
   const long long units = (long long)T * H;
   PSB_DISPATCH_DTYPE(gate_dtype, TG, {
     PSB_DISPATCH_DTYPE(out_dtype, TO, {
       psb_launch(normed_readout_kernel<TG, TO>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, stream, (const float*)o,
-                 (const TG*)gate, ldg, gate_act, (const float*)gain, (TO*)out, units, H, vdim, eps);
+                 (const TG*)gate, ldg, gate_act, (const float*)gain, head_gains, (TO*)out, ldo, units, H, vdim, eps);
     });
   });
   PSB_LAUNCH_CHECK("normed_readout");

@@ -46,6 +46,16 @@ def _ptr(t: torch.Tensor | None) -> int | None:
     return None if t is None else t.data_ptr()
 
 
+def _rows_out(out: torch.Tensor | None, rows: int, cols: int, dtype: torch.dtype, device: torch.device) -> tuple[torch.Tensor, int]:
+    """(the tensor a result of [rows, cols] goes to, its row stride): ``out``, which may be a run of columns of a wider
+    tensor, or a new one."""
+    if out is None:
+        out = torch.empty((rows, cols), dtype=dtype, device=device)
+    elif out.dim() != 2 or tuple(out.shape) != (rows, cols) or out.dtype != dtype or not out.is_cuda or (cols > 1 and out.stride(1) != 1):
+        raise KernelError(f"the result must go to {dtype} [{rows}, {cols}] with unit column stride, not {out.dtype} {tuple(out.shape)} strides {out.stride()}")
+    return out, max(int(out.stride(0)), cols)
+
+
 def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = None, scale: float = 1.0) -> torch.Tensor:
     """h[t] = float32(table[ids[t]]) * scale (the product in float32)."""
     _i32(ids, "token ids")
@@ -570,8 +580,9 @@ def gated_norm_add(h: torch.Tensor, y: torch.Tensor, gate: torch.Tensor | None, 
 UNARY_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "xielu": 2, "relu2": 3}  # the codes of activation.cu; xielu takes two learned numbers
 
 
-def activation(x: torch.Tensor, name: str, params: torch.Tensor | None = None) -> torch.Tensor:
-    """act(x) element by element; ``params``: float32 numbers of the activation on the device (xielu: p, q)."""
+def activation(x: torch.Tensor, name: str, params: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(x) element by element; ``params``: float32 numbers of the activation on the device (xielu: p, q).  ``out``: where
+    the rows of the result go (may be a run of columns of a wider tensor; x is then [T, W])."""
     try:
         code = UNARY_ACTIVATIONS[name]
     except KeyError:
@@ -580,10 +591,27 @@ def activation(x: torch.Tensor, name: str, params: torch.Tensor | None = None) -
     if name == "xielu":
         if params is None or params.dtype != torch.float32 or params.numel() != 2 or not params.is_cuda:
             raise KernelError("xielu needs its two numbers as float32 on the device")
-    out = torch.empty_like(x)
-    check(lib().psb_unary_act(x.data_ptr(), _code(x, "activation input"), out.data_ptr(), x.numel(), code, _ptr(params), _stream()),
+    if out is None:
+        out, cols, ld = torch.empty_like(x), max(x.numel(), 1), max(x.numel(), 1)
+    else:
+        cols = x.shape[-1]
+        out, ld = _rows_out(out, x.numel() // cols, cols, x.dtype, x.device)
+    check(lib().psb_unary_act(x.data_ptr(), _code(x, "activation input"), out.data_ptr(), x.numel(), cols, ld, code, _ptr(params), _stream()),
           "unary_act")
     return out
+
+
+def unary_linear(x: torch.Tensor, w: torch.Tensor, name: str, out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(x[M,K] @ w[N,K]^T) for an activation without numbers of its own.  bfloat16: in the product's epilogue where this
+    library runs the product (few rows, some dozens, many); otherwise product, then activation.  ``out``: where the rows of
+    the result go (may be a run of columns of a wider tensor)."""
+    if name in ACTIVATIONS and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
+        from .tensorcore import unary_linear_bf16
+        _dev(x, "left operand"), _dev(w, "weight")
+        out, ld = _rows_out(out, x.shape[0], w.shape[0], x.dtype, x.device)
+        if unary_linear_bf16(x, w, ACTIVATIONS[name], out, ld):
+            return out
+    return activation(linear(x, w), name, out=out)
 
 
 def latent_prepare(proj: torch.Tensor, positions: torch.Tensor, token_item: torch.Tensor, table: torch.Tensor,
@@ -896,12 +924,16 @@ def biased_attention(qkv: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, c
 
 def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, ctx, *, num_heads: int, num_kv_heads: int,
                         dim: int, vdim: int, page_size: int, scale: float, window: int | None = None, chunk: int | None = None,
-                        bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, keep_first: int = 0) -> torch.Tensor:
+                        bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, keep_first: int = 0,
+                        softcap: float | None = None, gate: torch.Tensor | None = None, out_scale: float = 1.0,
+                        out: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of queries [T, hq, dim] over a cache entry that holds one row per token and key/value head, the
     key and then the value ([pages, 1, hkv, page_size, dim + vdim]; the step's own rows already appended), with an
     optional window, chunk mask, distance bias (float32 [heads, reach]) and sink (float32 [heads]: a score per head
     that joins the softmax denominator without a value) -> [T, hq * vdim].  ``keep_first`` (with a window): the first so
-    many keys of a sequence stay visible to every later query."""
+    many keys of a sequence stay visible to every later query.  ``softcap``: the scaled scores pass softcap * tanh(s /
+    softcap) first.  The result is multiplied by ``out_scale`` and by sigmoid(``gate``) ([T, hq * vdim] in the queries' type,
+    rows may be runs of columns of a wider product) and goes to ``out``, which may be a run of columns as well."""
     keep_first = int(keep_first or 0)
     if keep_first and (not window or chunk):
         raise KernelError("kept first keys go with a window and no chunk mask")
@@ -919,7 +951,13 @@ def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, 
         reach = bias.shape[1]
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != num_heads or not sink.is_cuda):
         raise KernelError(f"sinks must be float32 [{num_heads}] on the device")
-    out = torch.empty((t, num_heads * vdim), dtype=q.dtype, device=q.device)
+    out, ldo = _rows_out(out, t, num_heads * vdim, q.dtype, q.device)
+    ldg = 0
+    if gate is not None:
+        if tuple(gate.shape) != (t, num_heads * vdim) or gate.dtype != q.dtype or not gate.is_cuda or (gate.shape[1] > 1 and gate.stride(1) != 1):
+            raise KernelError(f"the output gate must be {q.dtype} [{t}, {num_heads * vdim}] with unit column stride, is {gate.dtype} {tuple(gate.shape)}")
+        ldg = max(int(gate.stride(0)), num_heads * vdim)
+    tail = (_ptr(gate), ldg, ldo, float(out_scale), float(softcap or 0.0))
     win, chk = int(window or 0), int(chunk or 0)
     # Portions of a bfloat16 step go tile by tile; what is left (single tokens, short portions) walks its keys.  Which
     # kernel a token gets depends on the length of its portion only (decided on the device from the item offsets, so
@@ -939,9 +977,9 @@ def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, 
                                          table.data_ptr(), table.shape[1], positions.data_ptr(), token_item.data_ptr(),
                                          _ptr(bias), _ptr(sink), out.data_ptr(), t, num_heads, num_kv_heads, dim, vdim,
                                          page_size, win, chk, reach, float(scale), item_start.data_ptr(), 0, keep_first,
-                                         _ptr(partial), splits, _stream()), "attention_biased")
+                                         _ptr(partial), splits, *tail, _stream()), "attention_biased")
         return out
-    on_tensor_cores = both16 and BIASED_MMA and bool(lib().psb_attention_biased_mma_supported(num_heads, num_kv_heads, dim, vdim))
+    on_tensor_cores = both16 and BIASED_MMA and ldo % 2 == 0 and out.data_ptr() % 4 == 0 and bool(lib().psb_attention_biased_mma_supported(num_heads, num_kv_heads, dim, vdim))
     least = BIASED_MMA_MIN_TOKENS if on_tensor_cores else BIASED_TILE_MIN_TOKENS
     long_portions = both16 and ctx.max_new_tokens >= least
     tiled = long_portions and (on_tensor_cores or bool(lib().psb_attention_biased_tile_supported(num_heads, num_kv_heads, dim, vdim)))
@@ -950,12 +988,12 @@ def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, 
                                          table.data_ptr(), table.shape[1], positions.data_ptr(), token_item.data_ptr(),
                                          _ptr(bias), _ptr(sink), out.data_ptr(), t, num_heads, num_kv_heads, dim, vdim,
                                          page_size, win, chk, reach, float(scale), item_start.data_ptr(),
-                                         least if tiled else 0, keep_first, None, 1, _stream()), "attention_biased")
+                                         least if tiled else 0, keep_first, None, 1, *tail, _stream()), "attention_biased")
     if tiled:
         entry = lib().psb_attention_biased_mma if on_tensor_cores else lib().psb_attention_biased_tiles
         check(entry(q.data_ptr(), kv.data_ptr(), table.data_ptr(), table.shape[1], positions.data_ptr(), item_start.data_ptr(),
                     ctx.num_items, t, least, _ptr(bias), _ptr(sink), out.data_ptr(), num_heads, num_kv_heads, dim,
-                    vdim, page_size, win, chk, reach, float(scale), keep_first, _stream()),
+                    vdim, page_size, win, chk, reach, float(scale), keep_first, *tail, _stream()),
               "attention_biased_mma" if on_tensor_cores else "attention_biased_tiles")
     return out
 
@@ -1184,21 +1222,74 @@ def linear_attention(proj: torch.Tensor, alpha: torch.Tensor, state: torch.Tenso
     return o
 
 
+READOUT_GATES = {None: 0, "silu": 1, "sigmoid": 2}
+
+
 def normed_readout(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: float, *, gate_act: str | None,
-                   out_dtype: torch.dtype) -> torch.Tensor:
-    """o float32 [T, H, V] -> (gain * rmsnorm(o) over V) * gate (``gate_act`` None: as it is; "silu": silu(gate)), [T, H * V].
-    ``gate`` [T, H * V], rows may be runs of columns of a wider product."""
+                   out_dtype: torch.dtype, out: torch.Tensor | None = None) -> torch.Tensor:
+    """o float32 [T, H, V] -> (gain * rmsnorm(o) over V) * gate (``gate_act`` None: as it is; "silu": silu(gate); "sigmoid"),
+    [T, H * V].  ``gain`` float32 [V], shared by the heads, or [H * V].  ``gate`` [T, H * V] and ``out``: rows may be runs of
+    columns of a wider tensor."""
     _dev(o, "read-out")
     t, h, v = o.shape
     if o.dtype != torch.float32 or gate.dim() != 2 or tuple(gate.shape) != (t, h * v) or gate.stride(1) != 1 or not gate.is_cuda:
         raise KernelError(f"read-out must be float32 and its gate [{t}, {h * v}], are {o.dtype} and {tuple(gate.shape)}")
-    if gate_act not in (None, "silu"):
-        raise KernelError(f"gate activation {gate_act!r}: None or 'silu'")
-    _f32_vector(gain, v, "read-out gain")
-    out = torch.empty((t, h * v), dtype=out_dtype, device=o.device)
+    if gate_act not in READOUT_GATES:
+        raise KernelError(f"gate activation {gate_act!r}: one of {list(READOUT_GATES)}")
+    of_heads = h > 1 and gain.numel() == h * v
+    _f32_vector(gain, h * v if of_heads else v, "read-out gain")
+    out, ldo = _rows_out(out, t, h * v, out_dtype, o.device)
     check(lib().psb_normed_readout(o.data_ptr(), gate.data_ptr(), _code(gate, "read-out gate"), max(int(gate.stride(0)), h * v),
-                                   0 if gate_act is None else 1, gain.data_ptr(), out.data_ptr(), _code(out, "gated read-out"), t, h, v,
-                                   float(eps), _stream()), "normed_readout")
+                                   READOUT_GATES[gate_act], gain.data_ptr(), 1 if of_heads else 0, out.data_ptr(), _code(out, "gated read-out"),
+                                   ldo, t, h, v, float(eps), _stream()), "normed_readout")
+    return out
+
+
+MATRIX_MEMORY_CHUNK = 64     # tokens a chunk of the tensor-core form (as in matrix_memory.cu)
+MATRIX_MEMORY_CHUNKED = 24   # bfloat16 steps whose longest portion has this many tokens take that form, shorter ones go token by token
+
+
+def matrix_memory_blocks(dim: int, vdim: int) -> int:
+    """Runs of columns the state of a head is worked on in, each with its own copy of the normalizer and the exponent."""
+    return -(-vdim // (128 if dim <= 256 else 64 if dim <= 512 else 32))
+
+
+def matrix_memory_state(heads: int, dim: int, vdim: int) -> int:
+    """float32 numbers of a request's state: S, the normalizers, the exponents, rounded up to 16 bytes."""
+    blocks = matrix_memory_blocks(dim, vdim)
+    return -(-heads * (dim * vdim + blocks * dim + blocks) // 4) * 4
+
+
+def matrix_memory(proj: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, gain: torch.Tensor, state: torch.Tensor, ctx, *,
+                  heads: int, dim: int, vdim: int, cap: float, eps: float, out: torch.Tensor | None = None) -> torch.Tensor:
+    """The matrix memory with exponential gates over every portion of the step, its read-out normed per head, multiplied by
+    ``gain`` (float32 [heads * vdim]) and by the sigmoid of the output gate -> [T, heads * vdim].  proj [T, q | k | v | output
+    gate | input gates | forget gates] (rows may be runs of columns of a wider product); gate biases float32 [heads]; state
+    float32 [num_slots, ``matrix_memory_state``] (rows may be strided), read and brought up to date."""
+    t = proj.shape[0]
+    want = 2 * heads * (dim + vdim) + 2 * heads
+    if not proj.is_cuda or proj.dim() != 2 or proj.shape[1] < want or proj.stride(1) != 1:
+        raise KernelError(f"matrix memory: projection must be [T, >= {want}] on the device, is {tuple(proj.shape)}")
+    _f32_vector(bias_i, heads, "input gate bias"), _f32_vector(bias_f, heads, "forget gate bias"), _f32_vector(gain, heads * vdim, "read-out gain")
+    stride = _slot_rows(state, matrix_memory_state(heads, dim, vdim), "matrix memory state")
+    blocks, dev = matrix_memory_blocks(dim, vdim), proj.device
+    out, ldo = _rows_out(out, t, heads * vdim, proj.dtype, dev)
+    o32 = torch.empty((t, heads, vdim), dtype=torch.float32, device=dev) if blocks > 1 else None
+    ld = int(proj.stride(0)) if t > 1 else max(int(proj.stride(0)), proj.shape[1])
+    chunked = (proj.dtype == torch.bfloat16 and ctx.max_new_tokens >= MATRIX_MEMORY_CHUNKED and ld % 8 == 0 and proj.data_ptr() % 16 == 0
+               and out.data_ptr() % 4 == 0 and ldo % 2 == 0 and stride % 4 == 0 and state.data_ptr() % 16 == 0
+               and bool(lib().psb_matrix_memory_chunks_supported(dim, vdim)))
+    chunks, scratch = ctx.num_items, None
+    if chunked:
+        chunks = t // MATRIX_MEMORY_CHUNK + ctx.num_items
+        scratch = torch.empty(chunks * heads * (dim * vdim + dim + 3), dtype=torch.float32, device=dev)
+    check(lib().psb_matrix_memory(proj.data_ptr(), _code(proj, "projection output"), ld, bias_i.data_ptr(), bias_f.data_ptr(), gain.data_ptr(),
+                                  state.data_ptr(), stride, _i32(ctx.item_start, "item offsets").data_ptr(), _i32(ctx.slots, "slots").data_ptr(),
+                                  out.data_ptr(), ldo, _ptr(o32), _ptr(scratch), ctx.num_items, chunks, heads, dim, vdim, blocks,
+                                  state.shape[0], float(cap), float(eps), dim ** -0.5, _stream()), "matrix_memory_chunks" if chunked else "matrix_memory")
+    if o32 is not None:
+        gate = proj[:, 2 * heads * dim + heads * vdim: 2 * heads * (dim + vdim)]
+        normed_readout(o32, gate, gain, eps, gate_act="sigmoid", out_dtype=proj.dtype, out=out)
     return out
 
 
@@ -1276,6 +1367,82 @@ def attention_prepare_normed(proj: torch.Tensor, kv: torch.Tensor, table: torch.
                                              _code(kv, "cache entry"), q.data_ptr(), t, num_heads, num_kv_heads, dim, vdim, page_size,
                                              kv.shape[0], float(eps), 1 if split_planes else 0, _stream()), "attention_prepare_normed")
     return q
+
+
+def attention_prepare_heads(proj: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, ctx, *, num_heads: int, num_kv_heads: int,
+                            dim: int, vdim: int, page_size: int, gain_q: torch.Tensor, gain_k: torch.Tensor, eps: float,
+                            cos: torch.Tensor | None = None, sin: torch.Tensor | None = None, rotary_dim: int | None = None,
+                            interleaved: bool = False, split_planes: bool = False, bias: torch.Tensor | None = None,
+                            first: torch.Tensor | None = None, first_bias: torch.Tensor | None = None,
+                            share: torch.Tensor | None = None) -> torch.Tensor:
+    """One pass over the fused projection [T, q | k | v]: the biases (float32, one per column), an RMS norm over every query
+    and key head with a gain (float32 [dim] for the query heads, another for the key heads), the rotation of the first
+    ``rotary_dim`` elements by position, keys and values appended to the cache entry (layouts as in ``attention_prepare``).
+    ``first`` [T, hkv * vdim] (rows may be runs of columns): values of an earlier layer, with their biases; then the stored
+    value is (1 - share) v + share * first (``share``: one float32 number on the device).  Returns the queries [T, hq, dim]."""
+    t = proj.shape[0]
+    want = (num_heads + num_kv_heads) * dim + num_kv_heads * vdim
+    _dev(kv, "cache entry"), _i32(table, "page table")
+    if not proj.is_cuda or proj.dim() != 2 or proj.shape[1] != want or proj.stride(1) != 1:
+        raise KernelError(f"projection output must be [T, {want}] on the device (rows may be part of wider ones), is {tuple(proj.shape)}")
+    entry = (2, num_kv_heads, page_size, dim) if split_planes else (1, num_kv_heads, page_size, dim + vdim)
+    if kv.dim() != 5 or tuple(kv.shape[1:]) != entry:
+        raise KernelError(f"cache entry must be [pages, {', '.join(map(str, entry))}], is {tuple(kv.shape)}")
+    if bias is not None:
+        _f32_vector(bias, want, "projection bias")
+    _f32_vector(gain_q, dim, "query gain"), _f32_vector(gain_k, dim, "key gain")
+    rotary_dim, max_pos = dim if rotary_dim is None else int(rotary_dim), 0
+    if cos is not None:
+        if sin is None or cos.shape != sin.shape or cos.dtype != torch.float32 or sin.dtype != torch.float32 or cos.dim() != 2 \
+                or cos.shape[1] != rotary_dim // 2 or rotary_dim % 2 or not 2 <= rotary_dim <= dim:
+            raise KernelError(f"angle tables must be float32 [positions, {rotary_dim // 2}] for {rotary_dim} rotated elements of {dim}")
+        _dev(cos, "cosines"), _dev(sin, "sines")
+        max_pos = cos.shape[0]
+        if ctx.max_kv_len > max_pos:
+            raise KernelError(f"a position of this step ({ctx.max_kv_len - 1}) lies beyond the angle tables ({max_pos} positions)")
+    if first is not None:
+        if tuple(first.shape) != (t, num_kv_heads * vdim) or first.dtype != proj.dtype or not first.is_cuda or (first.shape[1] > 1 and first.stride(1) != 1):
+            raise KernelError(f"values to mix in must be {proj.dtype} [{t}, {num_kv_heads * vdim}] with unit column stride, are {first.dtype} {tuple(first.shape)}")
+        if share is None or share.dtype != torch.float32 or share.numel() != 1 or not share.is_cuda:
+            raise KernelError("the weight of the values that are mixed in must be one float32 number on the device")
+        if first_bias is not None:
+            _f32_vector(first_bias, num_kv_heads * vdim, "bias of the values that are mixed in")
+    q = torch.empty((t, num_heads, dim), dtype=proj.dtype, device=proj.device)
+    check(lib().psb_attention_prepare_heads(proj.data_ptr(), max(int(proj.stride(0)), want), _code(proj, "projection output"),
+                                            _i32(ctx.positions, "positions").data_ptr(), _i32(ctx.token_item, "token-to-item map").data_ptr(),
+                                            table.data_ptr(), table.shape[1], _ptr(cos), _ptr(sin), _ptr(bias), gain_q.data_ptr(),
+                                            gain_k.data_ptr(), _ptr(first), 0 if first is None else max(int(first.stride(0)), num_kv_heads * vdim),
+                                            _ptr(first_bias) if first is not None else None, _ptr(share) if first is not None else None,
+                                            kv.data_ptr(), _code(kv, "cache entry"), q.data_ptr(), t, num_heads, num_kv_heads, dim, vdim,
+                                            page_size, kv.shape[0], max_pos, rotary_dim, 1 if interleaved else 0, float(eps),
+                                            1 if split_planes else 0, _stream()), "attention_prepare_heads")
+    return q
+
+
+def add_layer_norm(h: torch.Tensor, pending: torch.Tensor | None, norms, eps: float, out_dtype: torch.dtype,
+                   rows: torch.Tensor | None = None) -> list[torch.Tensor]:
+    """h += pending (float32, in place, unless ``rows``); returns one or two layer norms of the result, a (gain, shift) pair
+    of float32 vectors each, for all or the chosen rows.  ``pending`` must have ``out_dtype``."""
+    _dev(h, "residual stream")
+    if h.dtype != torch.float32 or h.dim() != 2 or not 1 <= len(norms) <= 2:
+        raise KernelError(f"one or two layer norms of a float32 stream [T, W], not {len(norms)} of {h.dtype} {tuple(h.shape)}")
+    width, n = h.shape[1], h.shape[0]
+    if isinstance(pending, PendingProduct):
+        pending = pending.tensor()
+    if pending is not None:
+        _dev(pending, "sublayer output")
+        if pending.shape != h.shape or pending.dtype != out_dtype:
+            raise KernelError(f"sublayer output {pending.dtype} {tuple(pending.shape)} does not match the stream {tuple(h.shape)} in {out_dtype}")
+    if rows is not None:
+        n = _i32(rows, "row index").numel()
+    for gain, shift in norms:
+        _f32_vector(gain, width, "norm gain"), _f32_vector(shift, width, "norm shift")
+    xs = [torch.empty((n, width), dtype=out_dtype, device=h.device) for _ in norms]
+    second = norms[1] if len(norms) > 1 else (None, None)
+    check(lib().psb_add_layer_norm(h.data_ptr(), _ptr(pending), _code(xs[0], "normed rows"), norms[0][0].data_ptr(), norms[0][1].data_ptr(),
+                                   _ptr(second[0]), _ptr(second[1]), _ptr(rows), xs[0].data_ptr(), _ptr(xs[1]) if len(xs) > 1 else None,
+                                   n, width, float(eps), 1 if rows is None and pending is not None else 0, _stream()), "add_layer_norm")
+    return xs
 
 
 def poly_norm(z: torch.Tensor, act: torch.Tensor, eps: float) -> torch.Tensor:

@@ -132,8 +132,8 @@ _SIGNATURES: dict[str, list] = {
     "psb_hashed_embedding": [P, P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, L, L, I, P],
     # (h, y, y_dtype, g, g_dtype, bias, gain, copy, copy_dtype, rows, H, eps, mult, stream)
     "psb_gated_norm_add": [P, P, I, P, I, P, P, P, I, I, I, F, F, P],
-    # (x, dtype, out, total, code, params, stream)
-    "psb_unary_act": [P, I, P, L, I, P, P],
+    # (x, dtype, out, total, cols, ldo, code, params, stream)
+    "psb_unary_act": [P, I, P, L, L, L, I, P, P],
     # (x, x_dtype, gate_f32, out, out_dtype, total, stream)
     "psb_gate_mul": [P, I, P, P, I, L, P],
     # (proj, dtype, positions, token_item, table, table_width, cos, sin, gain_q, gain_kv, cq_out, gate_out, cache, cache_dtype,
@@ -169,14 +169,14 @@ _SIGNATURES: dict[str, list] = {
     "psb_attention_biased_append": [P, I, P, P, P, I, P, I, P, I, I, I, I, I, I, I, P],
     # (q, dtype, kv, kv_dtype, table, table_width, positions, token_item, bias, sink, out, T, hq, hkv, dim, vdim, page_size,
     #  window, chunk, reach, scale, item_start, skip_from, stream)
-    "psb_attention_biased": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, I, I, P, I, P],
+    "psb_attention_biased": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, I, I, P, I, P, L, L, F, F, P],
     "psb_attention_biased_tile_tokens": [],
     "psb_attention_biased_tile_supported": [I, I, I, I],
     # (q, kv, table, table_width, positions, item_start, items, T, min_tokens, bias, sink, out, hq, hkv, dim, vdim,
     #  page_size, window, chunk, reach, scale, stream)
-    "psb_attention_biased_tiles": [P, P, P, I, P, P, I, I, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P],
+    "psb_attention_biased_tiles": [P, P, P, I, P, P, I, I, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P, L, L, F, F, P],
     "psb_attention_biased_mma_supported": [I, I, I, I],
-    "psb_attention_biased_mma": [P, P, P, I, P, P, I, I, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P],
+    "psb_attention_biased_mma": [P, P, P, I, P, P, I, I, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P, L, L, F, F, P],
     "psb_delta_max_taps": [],
     # (proj, dtype, ld, beta_at, ba, decay, taps, a_log, dt_bias, state, positions, token_item, item_start, slots, qkv_out, bd_out, T,
     #  G, H, dim, vdim, K, num_slots, slot_floats, stream)
@@ -227,8 +227,23 @@ _SIGNATURES: dict[str, list] = {
     # (proj, dtype, ld, alpha, state, slot_floats, item_start, slots, local_b, local_a, o, items, chunks, H, dim, vdim, num_slots,
     #  chunk, scale, stream)
     "psb_linear_attention": [P, I, L, P, P, L, P, P, P, P, P, I, I, I, I, I, I, I, F, P],
-    # (o, gate, gate_dtype, ldg, gate_act, gain, out, out_dtype, T, H, vdim, eps, stream)
-    "psb_normed_readout": [P, P, I, L, I, P, P, I, I, I, I, F, P],
+    # (o, gate, gate_dtype, ldg, gate_act, gain, head_gains, out, out_dtype, ldo, T, H, vdim, eps, stream)
+    "psb_normed_readout": [P, P, I, L, I, P, I, P, I, L, I, I, I, F, P],
+    # (h, pending, dtype, gain1, shift1, gain2, shift2, rows, x1, x2, n_rows, W, eps, update, stream)
+    "psb_add_layer_norm": [P, P, I, P, P, P, P, P, P, P, I, I, F, I, P],
+    # (proj, ld, dtype, positions, token_item, table, table_width, cos, sin, bias, gain_q, gain_k, first, ld_first, first_bias, share,
+    #  kv, kv_dtype, q_out, T, hq, hkv, dim, vdim, page_size, num_pages, max_positions, rotary_dim, interleaved, eps, split_planes, stream)
+    "psb_attention_prepare_heads": [P, L, I, P, P, P, I, P, P, P, P, P, P, L, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+    # (proj, dtype, ld, bias_i, bias_f, gain, state, slot_floats, item_start, slots, out, ldo, o32, scratch, items, chunks, H, dim, vdim,
+    #  nb, num_slots, cap, eps, scale, stream)
+    "psb_matrix_memory": [P, I, L, P, P, P, P, L, P, P, P, L, P, P, I, I, I, I, I, I, I, F, F, F, P],
+    "psb_matrix_memory_chunks_supported": [I, I],
+    # (a, w, c, M, N, K, ldc, sms, activation, stream)
+    "psb_gemm_tcgen05_unary": [P, P, P, I, I, I, I, I, I, P],
+    # (x, W, y, M, N, K, ldy, sms, activation, stream)
+    "psb_gemm_stream_unary": [P, P, P, I, I, I, I, I, I, P],
+    # (a, w, c, M, N, K, ldc, activation, stream)
+    "psb_gemm_fewrows_unary": [P, P, P, I, I, I, I, I, P],
     # (proj, ld, dtype, positions, token_item, table, table_width, bias, gain, kv, kv_dtype, q_out, T, hq, hkv, dim, vdim, page_size,
     #  num_pages, eps, split_planes, stream)
     "psb_attention_prepare_normed": [P, L, I, P, P, P, I, P, P, P, I, P, I, I, I, I, I, I, I, F, I, P],

@@ -354,6 +354,27 @@ def linear_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> tor
     return y if out_dtype == y.dtype else y.to(out_dtype)
 
 
+def unary_linear_bf16(x: torch.Tensor, w: torch.Tensor, activation: int, out: torch.Tensor, ld: int) -> bool:
+    """act(x @ w^T) into ``out`` (rows ``ld`` numbers apart) with the activation in the product's epilogue, on whichever of
+    this library's products takes the shape (few rows, some dozens, many); False when none does and nothing has run."""
+    m, k = x.shape
+    n = w.shape[0]
+    if small_m_ok(m, k, min(STREAM_M, 16)):
+        check(lib().psb_gemm_stream_unary(x.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, ld, _sms(x.device), activation,
+                                          stream_handle()), "gemm_stream_unary")
+        return True
+    if out.data_ptr() % 16 or m == 0:
+        return False
+    if _fewrows_ok(x, w):
+        check(lib().psb_gemm_fewrows_unary(x.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, ld, activation, stream_handle()), "gemm_fewrows_unary")
+        return True
+    if m > STREAM_M and _tcgen05_ok(x, w):
+        check(lib().psb_gemm_tcgen05_unary(x.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, ld, _sms(x.device), activation,
+                                           stream_handle()), "gemm_tcgen05_unary")
+        return True
+    return False
+
+
 def gated_linear_bf16(x: torch.Tensor, w_gate_up: torch.Tensor, activation: int = 0) -> torch.Tensor | None:
     """act(x Wg^T) * (x Wu^T) in one kernel (few rows: the streaming product; many: the tcgen05 product); None when
     neither takes the shape."""

@@ -1,4 +1,4 @@
-from . import attention, biased_attention, combined, delta, embedding, ffn, gate, latent_attention, linear_attention, min_gru, moe, norm, normed_attention, position, recurrent, stream  # noqa: F401  (registers the built-in kinds)
+from . import attention, biased_attention, combined, delta, embedding, ffn, gate, head_norm_attention, latent_attention, linear_attention, matrix_memory, min_gru, moe, norm, normed_attention, position, recurrent, stream  # noqa: F401  (registers the built-in kinds)
 from .base import (CacheNeed, CacheView, FeedForward, FixedState, Gate, ItemView, Mixer, Norm, PagedKV, ParamSpec, Part,
                    PositionEncoding, StepContext)
 from .block import Block, register_arrangement

@@ -129,6 +129,19 @@ class Part:
     # ``ctx.items`` on the host must leave this False.
     graph_safe = False
 
+    # A mixer or feed-forward whose result is one matrix product of rows it has made may offer those rows instead: how many
+    # numbers a token they have (0: not offered).  ``forward_rows(x, ctx[, cache], out=...)`` then leaves them in ``out``
+    # [T, rows_width] (may be a run of columns of a wider tensor) and ``output_weight()`` is the matrix [H, rows_width] that
+    # the result is their product with.  Whoever adds the results of several such parts multiplies once, by the matrices
+    # side by side (see ``Block.join_outputs``); ``drop_output_weight()`` says that nobody asks for ``forward`` any more.
+    rows_width = 0
+
+    def output_weight(self) -> torch.Tensor:
+        raise NotImplementedError
+
+    def drop_output_weight(self) -> None:
+        raise NotImplementedError
+
     def __init__(self, spec_params: Mapping[str, Any]) -> None:
         self.params = dict(spec_params)
 

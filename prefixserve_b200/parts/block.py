@@ -9,6 +9,9 @@ h += scale_1 * mixer(x); h += scale_2 * ffn(x).
 ``parallel``: both sublayers read the same stream, h += mixer(norm_a(h)) + ffn(norm_b(h)).  Without a norm of its own
 (``ffn_norm`` None) the feed-forward reads the mixer's normed row, h += mixer(x) + ffn(x) with x = norm(h), and both
 results travel on together (``ops.StreamSum``) to the next norm's kernel.
+``parallel_rows``: h += mixer(norm_a(h)) + ffn(norm_b(h)) for sublayers that offer the rows their last products read
+(``Part.rows_width``): both leave them side by side in one tensor, and one product with the two matrices side by side is the
+sum of the results (rounded once, not twice).  The two norms share their statistics where they can (``LayerNorm.with_second``).
 ``gated_post_norm``: the sublayers read the stream itself and the norm sits on their result, behind a gate computed
 from the same input: h += scale * norm_a(mixer(h) * sigmoid(gate_a(h))); then the same with the feed-forward.
 
@@ -25,6 +28,8 @@ layer without feed-forward) and is added with ``register_arrangement``.
 from __future__ import annotations
 
 from typing import Callable
+
+import torch
 
 from .. import ops
 from ..config.spec import LayerSpec
@@ -57,6 +62,8 @@ class Block:
         self.ffn_post_norm = make("norm", spec.ffn_post_norm) if spec.ffn_post_norm is not None and spec.ffn is not None else None
         self.mixer_scale = make("gate", spec.mixer_scale) if spec.mixer_scale is not None else None
         self.ffn_scale = make("gate", spec.ffn_scale) if spec.ffn_scale is not None and spec.ffn is not None else None
+        self.w_out = None                # parallel_rows: the sublayers' last matrices side by side
+        self.row_columns: list[tuple[int, int]] = []
         if (self.mixer_scale is not None or self.ffn_scale is not None) and spec.arrangement != "pre_norm":
             raise ValueError("a channel scale on a sublayer's result goes with the pre_norm arrangement")
 
@@ -77,6 +84,26 @@ class Block:
             if self.ffn_scale is not None:
                 parts.append(("ffn_scale", self.ffn_scale))
         return tuple(parts)
+
+    def join_outputs(self) -> None:
+        """Called once the parts have their tensors: in the parallel_rows arrangement the last matrices of mixer and
+        feed-forward become one, each part's columns starting at a multiple of 8 (zeros fill the gaps)."""
+        if self.run is not parallel_rows:
+            return
+        parts = [self.mixer] + ([self.ffn] if self.ffn is not None else [])
+        if any(p.rows_width < 1 for p in parts):
+            raise ValueError("the parallel_rows arrangement needs sublayers that offer the rows their last product reads")
+        weights = [p.output_weight() for p in parts]
+        at = 0
+        for p in parts:
+            self.row_columns.append((at, at + p.rows_width))
+            at += -(-p.rows_width // 8) * 8
+        dtype = torch.float32 if any(w.dtype == torch.float32 for w in weights) else weights[0].dtype
+        self.w_out = torch.zeros((weights[0].shape[0], at), dtype=dtype, device=weights[0].device)
+        for w, (lo, hi) in zip(weights, self.row_columns):
+            self.w_out[:, lo:hi] = w
+        for p in parts:
+            p.drop_output_weight()
 
     def forward(self, h, pending, ctx: StepContext, cache: CacheView):
         return self.run(self, h, pending, ctx, cache)
@@ -114,6 +141,23 @@ def parallel(block: Block, h, pending, ctx: StepContext, cache: CacheView):
     fed = block.ffn.forward(block.ffn_norm.forward(h, None, ctx), ctx)
     ops.residual_add(h, mixed)
     return h, fed
+
+
+def parallel_rows(block: Block, h, pending, ctx: StepContext, cache: CacheView):
+    """Both sublayers see the stream as it entered the block; one product makes the sum of their results."""
+    pair = None
+    if block.ffn is not None and hasattr(block.mixer_norm, "with_second"):
+        pair = block.mixer_norm.with_second(block.ffn_norm, h, pending, ctx)
+    x = pair[0] if pair else block.mixer_norm.forward(h, pending, ctx)
+    used = sum(hi - lo for lo, hi in block.row_columns)
+    make_rows = torch.empty if used == block.w_out.shape[1] else torch.zeros  # nothing but numbers may meet the zeros of the gaps
+    rows = make_rows((h.shape[0], block.w_out.shape[1]), dtype=ctx.compute_dtype, device=h.device)
+    (lo, hi), *rest = block.row_columns
+    block.mixer.forward_rows(x, ctx, cache, out=rows[:, lo:hi])
+    if block.ffn is not None:
+        x = pair[1] if pair else block.ffn_norm.forward(h, None, ctx)
+        block.ffn.forward_rows(x, ctx, out=rows[:, rest[0][0]: rest[0][1]])
+    return h, ops.linear(rows, block.w_out)
 
 
 STREAM_COPY = "stream_in_compute_type"  # ctx.extras: (the stream tensor, its current value in the compute type)
@@ -165,3 +209,4 @@ register_arrangement("pre_norm", pre_norm)
 register_arrangement("sandwich_norm", sandwich_norm)
 register_arrangement("gated_post_norm", gated_post_norm)
 register_arrangement("parallel", parallel)
+register_arrangement("parallel_rows", parallel_rows)

@@ -10,7 +10,11 @@ their input (they offer ``input_weight`` / ``forward_projected``) share a single
 With ``deferred_sum`` the two results are handed on as they are (``ops.NormedPair``) and the norm in front of the next
 sublayer does both norms and the sums in its own kernel; only for arrangements whose norms take one.
 
-Both hand their inner mixers' tensors, paged cache need and graph-safety through.  Fixed states are float32 vectors
+``side_by_side_sum``: the same without the norms, for branches that offer the rows their last product reads
+(``Part.rows_width``): their rows lie side by side and one product with the two matrices side by side is the sum of the
+results.  A factor on a branch's result is that branch's own (``out_scale``).
+
+All hand their inner mixers' tensors, paged cache need and graph-safety through.  Fixed states are float32 vectors
 laid one after the other in the slot's state (the combinator's own first); an inner mixer sees its run of columns,
 so its kernels must take a state whose rows are part of wider ones (the row stride is the tensor's).
 """
@@ -88,23 +92,23 @@ class TokenShifted(Mixer):
         return self.inner.forward(shifted, ctx, _inner_view(cache, self.inner_need, self.size, self.inner_floats, alone=False))
 
 
-class SideBySide(Mixer):
+class _Branches(Mixer):
+    """Two mixers on the same input: their tensors, cache need, state columns, and one product for the matrices both apply
+    to their input first."""
+
     def __init__(self, params):
         super().__init__(params)
         self.hidden = int(params["hidden_size"])
-        self.eps = float(params["eps"])
         self.names = tuple(str(n) for n in params.get("names") or ("left", "right"))
         self.branches = [make("mixer", _as_spec(s)) for s in params["branches"]]
+        kind = type(self).__name__
         if len(self.branches) != 2 or len(self.names) != 2:
-            raise ValueError("side_by_side is built for two branches")  # the kernel that norms and adds takes a pair
-        self.weight = float(params.get("weight", 1.0 / len(self.branches)))
-        self.deferred_sum = bool(params.get("deferred_sum", False))
+            raise ValueError(f"{kind} is built for two branches")
         self.needs = [b.cache_need() for b in self.branches]
         if sum(n.paged is not None for n in self.needs) > 1:
-            raise ValueError("side_by_side: at most one branch may keep keys and values (a cache entry has one set of pages)")
-        self.floats = [_state_floats(n, "side_by_side") for n in self.needs]
+            raise ValueError(f"{kind}: at most one branch may keep keys and values (a cache entry has one set of pages)")
+        self.floats = [_state_floats(n, kind) for n in self.needs]
         self.alone = sum(f > 0 for f in self.floats) == 1  # a single state passes through in its own shape
-        self.gains: list[torch.Tensor] = []
         self.w_in: torch.Tensor | None = None
         self.columns: list[tuple[int, int]] = []
 
@@ -116,8 +120,6 @@ class SideBySide(Mixer):
         specs = {}
         for name, b in zip(self.names, self.branches):
             specs.update({f"{name}.{local}": ps for local, ps in b.param_specs().items()})
-        for name in self.names:
-            specs[f"{name}_gain"] = ParamSpec((self.hidden,), role="vector", init="ones")
         return specs
 
     def cache_need(self):
@@ -131,7 +133,6 @@ class SideBySide(Mixer):
     def load(self, tensors, *, compute_dtype, device):
         for name, b in zip(self.names, self.branches):
             b.load({k[len(name) + 1:]: t for k, t in tensors.items() if k.startswith(name + ".")}, compute_dtype=compute_dtype, device=device)
-        self.gains = [tensors[f"{name}_gain"].to(device=device, dtype=torch.float32).contiguous() for name in self.names]
         # one product for every branch that starts with a matrix of its own on the shared input
         if all(hasattr(b, "input_weight") and hasattr(b, "forward_projected") for b in self.branches):
             pieces = [b.input_weight() for b in self.branches]
@@ -148,12 +149,36 @@ class SideBySide(Mixer):
         for b in self.branches:
             b.prepare(max_positions=max_positions, compute_dtype=compute_dtype, device=device)
 
+    def views(self, cache: CacheView):
+        """The cache entry as each branch sees it."""
+        at = 0
+        for need, floats in zip(self.needs, self.floats):
+            yield _inner_view(cache, need, at, floats, alone=self.alone)
+            at += floats
+
+
+class SideBySide(_Branches):
+    def __init__(self, params):
+        super().__init__(params)
+        self.eps = float(params["eps"])
+        self.weight = float(params.get("weight", 1.0 / len(self.branches)))
+        self.deferred_sum = bool(params.get("deferred_sum", False))
+        self.gains: list[torch.Tensor] = []
+
+    def param_specs(self):
+        specs = super().param_specs()
+        for name in self.names:
+            specs[f"{name}_gain"] = ParamSpec((self.hidden,), role="vector", init="ones")
+        return specs
+
+    def load(self, tensors, *, compute_dtype, device):
+        super().load(tensors, compute_dtype=compute_dtype, device=device)
+        self.gains = [tensors[f"{name}_gain"].to(device=device, dtype=torch.float32).contiguous() for name in self.names]
+
     def forward(self, x, ctx: StepContext, cache: CacheView):
         proj = ops.linear(x, self.w_in) if self.w_in is not None else None
-        results, at = [], 0
-        for i, (b, need) in enumerate(zip(self.branches, self.needs)):
-            view = _inner_view(cache, need, at, self.floats[i], alone=self.alone)
-            at += self.floats[i]
+        results = []
+        for i, (b, view) in enumerate(zip(self.branches, self.views(cache))):
             if proj is not None:
                 lo, hi = self.columns[i]
                 y = b.forward_projected(proj[:, lo:hi], ctx, view)
@@ -165,5 +190,50 @@ class SideBySide(Mixer):
         return ops.normed_pair_sum(results[0], results[1], self.gains[0], self.gains[1], self.eps, self.weight)
 
 
+class SideBySideSum(_Branches):
+    def __init__(self, params):
+        super().__init__(params)
+        if any(b.rows_width < 1 or not hasattr(b, "forward_rows_projected") for b in self.branches):
+            raise ValueError("side_by_side_sum needs branches that offer the rows their last product reads")
+        self.starts = [0, -(-self.branches[0].rows_width // 8) * 8]  # the second branch's rows start on 16 bytes
+        self.w_o: torch.Tensor | None = None
+
+    @property
+    def rows_width(self) -> int:
+        return self.starts[1] + self.branches[1].rows_width
+
+    def load(self, tensors, *, compute_dtype, device):
+        super().load(tensors, compute_dtype=compute_dtype, device=device)
+        if self.w_in is None:
+            raise ValueError("side_by_side_sum: the branches' input matrices are of different types")
+        weights = [b.output_weight() for b in self.branches]
+        dtype = torch.float32 if any(w.dtype == torch.float32 for w in weights) else weights[0].dtype
+        self.w_o = torch.zeros((self.hidden, self.rows_width), dtype=dtype, device=weights[0].device)
+        for w, at in zip(weights, self.starts):
+            self.w_o[:, at: at + w.shape[1]] = w
+        for b in self.branches:
+            b.drop_output_weight()
+
+    def output_weight(self):
+        return self.w_o
+
+    def drop_output_weight(self):
+        self.w_o = None
+
+    def forward_rows(self, x, ctx: StepContext, cache: CacheView, *, out):
+        proj = ops.linear(x, self.w_in)
+        first = self.branches[0].rows_width
+        if first < self.starts[1]:
+            out[:, first: self.starts[1]].zero_()  # meets zeros of the matrix
+        for b, view, (lo, hi), at in zip(self.branches, self.views(cache), self.columns, self.starts):
+            b.forward_rows_projected(proj[:, lo:hi], ctx, view, out=out[:, at: at + b.rows_width])
+
+    def forward(self, x, ctx: StepContext, cache: CacheView):
+        rows = torch.empty((x.shape[0], self.rows_width), dtype=x.dtype, device=x.device)
+        self.forward_rows(x, ctx, cache, out=rows)
+        return ops.linear(rows, self.w_o)
+
+
 register_mixer("token_shift", TokenShifted, replace=True)
 register_mixer("side_by_side", SideBySide, replace=True)
+register_mixer("side_by_side_sum", SideBySideSum, replace=True)

@@ -88,6 +88,19 @@ class DenseMLP(FeedForward):
         if self.learned:
             self.act_params = tensors["act"].to(device=device, dtype=torch.float32).contiguous()
 
+    @property
+    def rows_width(self) -> int:
+        return 0 if self.learned else self.inter
+
+    def output_weight(self):
+        return self.w_down
+
+    def drop_output_weight(self):
+        self.w_down = None
+
+    def forward_rows(self, x, ctx: StepContext, *, out):
+        ops.unary_linear(x, self.w_up, self.activation, out=out)
+
     def forward(self, x, ctx: StepContext):
         if self.activation == "poly_norm":
             return ops.linear(ops.poly_norm(ops.linear(x, self.w_up), self.act_params, self.eps), self.w_down)

@@ -53,6 +53,8 @@ class DecoderModel:
             mine = {local: tensors[f"{prefix}.{local}"] for local in p.param_specs()}
             p.load(mine, compute_dtype=compute_dtype, device=device)
             p.prepare(max_positions=max_positions, compute_dtype=compute_dtype, device=device)
+        for block in self.blocks:
+            block.join_outputs()
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding.table)
         self.compute_dtype = compute_dtype
@@ -63,7 +65,7 @@ class DecoderModel:
         tables that are not in the checkpoint (rotary angles) are not weights and do not count."""
         seen: set[int] = set()
         total = 0
-        for _, part in self.named_parts():
+        for part in [p for _, p in self.named_parts()] + self.blocks:  # (a block holds matrices it has put side by side)
             for value in vars(part).values():
                 if isinstance(value, torch.Tensor) and value.data_ptr() not in seen:
                     seen.add(value.data_ptr())

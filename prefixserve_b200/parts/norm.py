@@ -1,4 +1,4 @@
-"""RMSNorm, fused with the residual sum that precedes it.
+"""RMSNorm (and layer norm), fused with the residual sum that precedes it.
 
 y = gain * (x * rsqrt(mean(x^2) + eps)), everything in float32
 (prefixserve/model/llama.py:63-69).  The residual stream is float32; the
@@ -58,4 +58,35 @@ class RMSNorm(Norm):
         return ops.NormedRows(h, delta, self.gain, self.eps, ctx.compute_dtype, rows)
 
 
+class LayerNorm(Norm):
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias, everything in float32, fused with the residual sum in
+    front of it.  Two such norms of one stream (``with_second``) share the sum, the mean and the variance."""
+
+    graph_safe = True  # device work depends only on tensor shapes and device-side inputs
+
+    def __init__(self, params):
+        super().__init__(params)
+        self.size = int(params["size"])
+        self.eps = float(params["eps"])
+        self.gain: torch.Tensor | None = None
+        self.shift: torch.Tensor | None = None
+
+    def param_specs(self):
+        return {"weight": ParamSpec((self.size,), role="vector", init="ones"), "bias": ParamSpec((self.size,), role="vector", init="normal")}
+
+    def load(self, tensors, *, compute_dtype, device):
+        self.gain, self.shift = (tensors[n].to(device=device, dtype=torch.float32).contiguous() for n in ("weight", "bias"))
+
+    def forward(self, h, delta, ctx: StepContext, rows=None):
+        return ops.add_layer_norm(h, delta, [(self.gain, self.shift)], self.eps, ctx.compute_dtype, rows)[0]
+
+    def with_second(self, other: Norm, h, delta, ctx: StepContext):
+        """(this norm, another one) of the stream after ``delta`` has joined it, in one kernel; None when the two cannot
+        share their statistics."""
+        if not isinstance(other, LayerNorm) or other.eps != self.eps or other.size != self.size:
+            return None
+        return ops.add_layer_norm(h, delta, [(self.gain, self.shift), (other.gain, other.shift)], self.eps, ctx.compute_dtype)
+
+
 register_norm("rms", RMSNorm, replace=True)
+register_norm("layer", LayerNorm, replace=True)

@@ -10,6 +10,7 @@ With ``yarn`` scaling (factor, original_max_positions, fast, slow) the pair inde
 over the original length is d(t) = D ln(original / (2 pi t)) / (2 ln theta); pairs below lo = max(floor(d(fast)), 0)
 keep their frequency, pairs above hi = min(ceil(d(slow)), D - 1) have it divided by ``factor``, with a linear ramp
 between (clamp((j - lo) / max(hi - lo, 0.001), 0, 1)); cosines and sines are multiplied by 0.1 ln(factor) + 1.
+With ``linear`` scaling every frequency is divided by ``factor``.
 ``none``: no rotation; queries and keys go through unchanged.
 
 What a rotating part tells its mixer: ``cos``/``sin`` float32 [positions,
@@ -53,8 +54,10 @@ def rope_inverse_frequencies(head_dim: int, theta: float, scaling) -> torch.Tens
         hi = min(math.ceil(pair_of(float(scaling["slow"]))), head_dim - 1)
         ramp = ((torch.arange(head_dim // 2, dtype=torch.float32) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
         return inv / factor * ramp + inv * (1 - ramp)
+    if kind == "linear":
+        return inv / float(scaling["factor"])
     if kind != "llama3":
-        raise ValueError(f"rope scaling kind {kind!r} is not built (llama3, yarn)")
+        raise ValueError(f"rope scaling kind {kind!r} is not built (linear, llama3, yarn)")
     factor = float(scaling["factor"])
     low, high = float(scaling["low_freq_factor"]), float(scaling["high_freq_factor"])
     original = float(scaling["original_max_positions"])
