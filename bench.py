@@ -777,7 +777,11 @@ ZOMOLIX_SIZES = {"2048": ("zomolix-2048", "gekopel-2048"), "4096": ("zomolix-409
 # bounded span of keys read from a row per token, routed experts with a shared one), at the same width, sizes and number of
 # layer runs
 BUMALIX_SIZES = {"2048": ("bumalix-2048", "gekopel-2048"), "4096": ("bumalix-4096", "gekopel-4096")}
-BESIDE = {"nerenex": "llama", "gekopel": "nerenex", "goganex": "llama", "zomolix": "gekopel", "bumalix": "gekopel"}
+# --workload dogotar: the closest model already here is Bumalix (mixer and feed-forward side by side on one stream, attention with
+# biases and normed queries and keys over a bounded span of keys read from a row per token, beside a recurrence with a matrix
+# state), at the same width, heads, spans and number of layer runs
+DOGOTAR_SIZES = {"2048": ("dogotar-2048", "bumalix-2048"), "4096": ("dogotar-4096", "bumalix-4096")}
+BESIDE = {"nerenex": "llama", "gekopel": "nerenex", "goganex": "llama", "zomolix": "gekopel", "bumalix": "gekopel", "dogotar": "bumalix"}
 
 
 def run_nerenex(args, design: str = "nerenex") -> dict:
@@ -795,7 +799,10 @@ def run_nerenex(args, design: str = "nerenex") -> dict:
     a shared one; a learned scale per channel on every sublayer) beside Gekopel at the same width.
     --workload bumalix: the same for the Bumalix design (delta rule with a decay per key channel; windowed attention beside
     gated linear attention, twice; routed experts weighted on their input; a repeated run of layers mixed with the
-    embedding output) beside Gekopel at the same width and number of layer runs."""
+    embedding output) beside Gekopel at the same width and number of layer runs.
+    --workload dogotar: the same for the Dogotar design (windowed attention with normed heads, capped scores, value mixing and an
+    output gate; then, twice, chunked attention beside a matrix memory with exponential gates; dense feed-forward beside every
+    mixer) beside Bumalix at the same width and number of layer runs."""
     import re
 
     import numpy as np
@@ -808,7 +815,7 @@ def run_nerenex(args, design: str = "nerenex") -> dict:
 
     prompt, context, batches = 2048, args.context if "--context" in sys.argv else 2048, (8, 32)
     steps, warmup = min(args.steps, 32), max(3, min(args.warmup, 8))
-    sizes = {"gekopel": GEKOPEL_SIZES, "goganex": GOGANEX_SIZES, "zomolix": ZOMOLIX_SIZES, "bumalix": BUMALIX_SIZES}.get(design, NERENEX_SIZES)
+    sizes = {"gekopel": GEKOPEL_SIZES, "goganex": GOGANEX_SIZES, "zomolix": ZOMOLIX_SIZES, "bumalix": BUMALIX_SIZES, "dogotar": DOGOTAR_SIZES}.get(design, NERENEX_SIZES)
     out = {"workload": design, "dtype": "bf16", "data": "synthetic", "prompt": prompt, "context": context, "steps": steps,
            "warmup": warmup, "timing": "CUDA events; weights of every model exceed L2", "peaks": peaks(), "sizes": {}}
     for size in ([args.model] if args.model in sizes else sorted(sizes)):
@@ -819,7 +826,7 @@ def run_nerenex(args, design: str = "nerenex") -> dict:
             if which == design:
                 cfg = preset(own_name)
                 vocab = cfg.vocab
-            elif which in ("nerenex", "gekopel"):
+            elif which in ("nerenex", "gekopel", "bumalix"):
                 cfg = preset(llama_name)
                 vocab = cfg.vocab
             else:
@@ -966,12 +973,13 @@ def main() -> int:
     p.add_argument("--profile", action="store_true",
                    help="--timeline plus, per kernel, the bytes and flops it has to do in the step and the fraction of the "
                         "measured peak that its time inside the step amounts to")
-    p.add_argument("--workload", choices=["decode", "shared-prefix", "mixed", "nerenex", "gekopel", "goganex", "zomolix", "bumalix"], default="decode",
+    p.add_argument("--workload", choices=["decode", "shared-prefix", "mixed", "nerenex", "gekopel", "goganex", "zomolix", "bumalix", "dogotar"], default="decode",
                    help="decode: the headline line.  shared-prefix: 64 requests over 4 system prefixes through the entry "
                         "point, prefix cache on and off.  mixed: steps of one 512-token prompt portion beside 64 decoded tokens.  "
                         "nerenex: prefill and decode of the Nerenex design beside a Llama of the same width and depth (--model 2048|4096).  "
                         "gekopel: the same for the Gekopel design beside Nerenex.  goganex: the same for the Goganex design beside a Llama.  "
-                        "zomolix: the same for the Zomolix design beside Gekopel.  bumalix: the same for the Bumalix design beside Gekopel")
+                        "zomolix: the same for the Zomolix design beside Gekopel.  bumalix: the same for the Bumalix design beside Gekopel.  dogotar: the same for the "
+                        "Dogotar design beside Bumalix")
     p.add_argument("--model", choices=sorted(SIZES) + sorted(NERENEX_SIZES), default=None,
                    help="layer sizes for --workload shared-prefix (8b) / mixed (3b), and for --only decode (the headline stays 1b)")
     p.add_argument("--requests", type=int, default=64, help="requests of --workload shared-prefix")
@@ -1007,7 +1015,7 @@ def main() -> int:
             return 0
         if _no_device(args):
             return 1
-        if args.workload in ("nerenex", "gekopel", "goganex", "zomolix", "bumalix"):
+        if args.workload in ("nerenex", "gekopel", "goganex", "zomolix", "bumalix", "dogotar"):
             result = run_nerenex(args, args.workload)
             print(json.dumps(result))
             return 0
