@@ -24,6 +24,9 @@
 // Scores, weights and sums are float32 and the weights are not rounded before they multiply the values.  Float32 and
 // bfloat16 storage.
 //
+// attention_rows_single_kernel (bfloat16 storage, steps of single tokens): all query heads of a key/value head in one block, the
+// scores and the weighted sum on the tensor cores.
+//
 // attention_biased_tile_kernel (bfloat16 storage): a block takes 16 consecutive tokens of one request and one
 // key/value head, with all the query heads that share it; key/value rows are staged in shared memory once for the
 // block, a warp takes (token, head) pairs in turn and walks all runs of its pair in order.
@@ -688,6 +691,223 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   }
 }
 
+// Steps of single tokens in bfloat16 on the tensor cores: a block of four warps takes a token, a key/value head with up to 16 of
+// the query heads that read it, and a share of the keys.  Keys come in runs of 16 aligned to absolute positions; run r goes to
+// share (r / 4) mod splits, warp r mod 4, and every warp brings its own runs in with cp.async through a ring of its own, whole
+// cache rows (key, then value) at a time; a row outside the masks is zeros.  S = Q K^T (mma.sync m16n8k16: heads in rows, keys in
+// columns) stays in registers, where scale, cap, bias, masks and the online softmax are applied in float32; the weights enter the
+// second product as the sum of two bfloat16 numbers.  The warps are joined in warp order; with several shares the merge kernel
+// above joins them.
+constexpr int ROWS_WARPS = 4, ROWS_RUN = 16, ROWS_HEADS = 16, ROWS_STAGES = 3;
+
+__device__ __forceinline__ void rows_ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rows_ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rows_copy16(uint32_t dst, const void* src, bool there) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(there ? 16 : 0) : "memory");
+}
+
+// elements between the rows of a ring: an odd number of 16-byte pieces, so that ldmatrix meets every bank once
+__host__ __device__ __forceinline__ int rows_pitch(int row) { return (row / 8) % 2 ? row : row + 8; }
+inline size_t rows_smem(int dim, int vdim) {
+  const size_t ring = (size_t)ROWS_WARPS * ROWS_STAGES * ROWS_RUN * rows_pitch(dim + vdim) * 2 + 32;
+  const size_t join = (size_t)ROWS_WARPS * ROWS_HEADS * (vdim + 2) * 4;
+  return ring > join ? ring : join;
+}
+
+template <int D, int V>  // key and value sizes rounded up to 64 or 128
+__global__ void __launch_bounds__(ROWS_WARPS * 32)
+attention_rows_single_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kv, const int32_t* __restrict__ table,
+                             int table_width, const int32_t* __restrict__ positions, const int32_t* __restrict__ token_item,
+                             const float* __restrict__ bias, const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int hq, int hkv,
+                             int dim, int vdim, int page_size, int window, int chunk, int reach, float scale, int keep_first,
+                             float* __restrict__ partial, int splits, const RowsTail tail) {
+  extern __shared__ __align__(16) unsigned char rows_raw[];
+  pdl_trigger();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int share = hq / hkv, groups = (share + ROWS_HEADS - 1) / ROWS_HEADS;
+  const int t = blockIdx.x / (hkv * groups), rest = blockIdx.x - t * hkv * groups;
+  const int g = rest / groups, h0 = g * share + (rest - g * groups) * ROWS_HEADS;
+  const int heads = min(ROWS_HEADS, (g + 1) * share - h0);
+  // inputs of the step: they may be read before the preceding kernel has finished
+  const int p = positions[t];
+  const int32_t* pages = table + (size_t)token_item[t] * table_width;
+  int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+  if (chunk > 0) lo = max(lo, (p / chunk) * chunk);
+  int kept_runs = 0;  // kept first keys: one stretch from 0 while the window reaches them, else runs of their own in front
+  if (keep_first > 0) {
+    if (lo <= keep_first) lo = 0;
+    else kept_runs = (keep_first + ROWS_RUN - 1) / ROWS_RUN;
+  }
+  const int first_run = lo / ROWS_RUN, runs = kept_runs + p / ROWS_RUN - first_run + 1;
+  const int rw = dim + vdim, pitch = rows_pitch(rw), pieces = rw / 8;
+  const size_t head_stride = (size_t)page_size * rw, page_elems = (size_t)hkv * head_stride;
+  const uint32_t ring = (uint32_t)__cvta_generic_to_shared(rows_raw) + (uint32_t)(warp * ROWS_STAGES * ROWS_RUN * pitch * 2);
+  const int step = ROWS_WARPS * splits, mine = blockIdx.y * ROWS_WARPS + warp;
+  auto base_of = [&](int run) { return ROWS_RUN * (run < kept_runs ? run : first_run + run - kept_runs); };
+  pdl_wait();  // queries and this step's cache rows are the preceding kernels' output
+
+  auto fetch = [&](int run, int stage) {
+    if (run < runs) {
+      const int base = base_of(run);
+      long long off = -1;  // lane r: where row r of the run lies
+      if (lane < ROWS_RUN) {
+        const int key = base + lane;
+        if (run < kept_runs ? key < keep_first : (key >= lo && key <= p))
+          off = (long long)((size_t)pages[key / page_size] * page_elems + (size_t)g * head_stride + (size_t)(key % page_size) * rw);
+      }
+      const uint32_t dst = ring + (uint32_t)(stage * ROWS_RUN * pitch * 2);
+#pragma unroll 4
+      for (int r = 0; r < ROWS_RUN; ++r) {
+        const long long at = __shfl_sync(0xffffffffu, off, r);
+        for (int c = lane; c < pieces; c += 32) rows_copy16(dst + (uint32_t)(r * pitch + c * 8) * 2, kv + (at < 0 ? 0 : at) + c * 8, at >= 0);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int s = 0; s < ROWS_STAGES - 1; ++s) fetch(mine + s * step, s);
+
+  // the heads' queries as operand fragments (rows beyond the heads are zeros)
+  uint32_t qf[D / 16][4];
+#pragma unroll
+  for (int kk = 0; kk < D / 16; ++kk)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = gid + 8 * (e & 1), c = kk * 16 + 2 * tig + 8 * (e >> 1);
+      qf[kk][e] = row < heads && c < dim ? *reinterpret_cast<const uint32_t*>(q + ((size_t)t * hq + h0 + row) * dim + c) : 0u;
+    }
+  float m[2] = {-FLT_MAX, -FLT_MAX}, l[2] = {0.f, 0.f};
+  float o[V / 8][4];
+#pragma unroll
+  for (int i = 0; i < V / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  const int lrow = lane & 7, lmat = lane >> 3;
+  int stage = 0;
+  for (int run = mine; run < runs; run += step) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(ROWS_STAGES - 2) : "memory");
+    __syncwarp();  // every lane's copies of this run have landed, and every lane is done with the run before
+    fetch(run + (ROWS_STAGES - 1) * step, stage == 0 ? ROWS_STAGES - 1 : stage - 1);
+    const uint32_t src = ring + (uint32_t)(stage * ROWS_RUN * pitch * 2);
+    stage = stage + 1 == ROWS_STAGES ? 0 : stage + 1;
+    float sc[2][4] = {};
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      if (kk * 16 >= dim) break;
+      uint32_t b[4];
+      rows_ldmatrix4(b, src + (uint32_t)(((lmat >> 1) * 8 + lrow) * pitch + kk * 16 + (lmat & 1) * 8) * 2);
+      mma_16816(sc[0], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[0], b[1]);
+      mma_16816(sc[1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[2], b[3]);
+    }
+    const bool kept = run < kept_runs;
+    const int base = base_of(run);
+    float top[2] = {-FLT_MAX, -FLT_MAX};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = e >> 1, key = base + n * 8 + 2 * tig + (e & 1);
+        float v = sc[n][e] * scale;
+        if (tail.softcap > 0.f) v = tail.softcap * tanhf(v / tail.softcap);
+        if (bias && gid + 8 * r < heads) v += bias[(size_t)(h0 + gid + 8 * r) * reach + max(0, min(p - key, reach - 1))];
+        if (!(kept ? key < keep_first : (key >= lo && key <= p))) v = -INFINITY;
+        sc[n][e] = v;
+        top[r] = fmaxf(top[r], v);
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
+      top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
+      const float m_new = fmaxf(m[r], top[r]), alpha = expf(m[r] - m_new);
+      m[r] = m_new;
+      l[r] *= alpha;
+#pragma unroll
+      for (int i = 0; i < V / 8; ++i) { o[i][2 * r] *= alpha; o[i][2 * r + 1] *= alpha; }
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        sc[n][e] = expf(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
+        l[e >> 1] += sc[n][e];
+      }
+    uint32_t hi[4], lo4[4];
+    split_bf16(sc[0][0], sc[0][1], hi[0], lo4[0]);
+    split_bf16(sc[0][2], sc[0][3], hi[1], lo4[1]);
+    split_bf16(sc[1][0], sc[1][1], hi[2], lo4[2]);
+    split_bf16(sc[1][2], sc[1][3], hi[3], lo4[3]);
+#pragma unroll
+    for (int nv = 0; nv < V / 8; nv += 2) {
+      if (nv * 8 >= vdim) break;
+      uint32_t b[4];  // (values in an odd number of eights: the last columns read 16 bytes beyond the row, and nobody stores them)
+      rows_ldmatrix4_trans(b, src + (uint32_t)(((lmat & 1) * 8 + lrow) * pitch + dim + nv * 8 + (lmat >> 1) * 8) * 2);
+      mma_16816(o[nv], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+      mma_16816(o[nv], lo4[0], lo4[1], lo4[2], lo4[3], b[0], b[1]);
+      mma_16816(o[nv + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+      mma_16816(o[nv + 1], lo4[0], lo4[1], lo4[2], lo4[3], b[2], b[3]);
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+  }
+  __syncthreads();  // every warp has left its ring: the shares take its place, [warp][head][vdim | m | l]
+  float* join = reinterpret_cast<float*>(rows_raw);
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int row = gid + 8 * r;
+    if (row >= heads) continue;
+    float* dst = join + ((size_t)warp * ROWS_HEADS + row) * (vdim + 2);
+#pragma unroll
+    for (int i = 0; i < V / 8; ++i) {
+      const int c = i * 8 + 2 * tig;
+      if (c < vdim) { dst[c] = o[i][2 * r]; dst[c + 1] = o[i][2 * r + 1]; }
+    }
+    if (tig == 0) { dst[vdim] = m[r]; dst[vdim + 1] = l[r]; }
+  }
+  __syncthreads();
+  for (int row = warp; row < heads; row += ROWS_WARPS) {  // a warp a head
+    const int h = h0 + row;
+    const bool sink_here = sink && splits == 1;
+    float M = sink_here ? sink[h] : -FLT_MAX;
+    float mw[ROWS_WARPS], f[ROWS_WARPS];
+#pragma unroll
+    for (int w = 0; w < ROWS_WARPS; ++w) {
+      mw[w] = join[((size_t)w * ROWS_HEADS + row) * (vdim + 2) + vdim];
+      M = fmaxf(M, mw[w]);
+    }
+    float L = sink_here ? expf(sink[h] - M) : 0.f;
+#pragma unroll
+    for (int w = 0; w < ROWS_WARPS; ++w) {
+      f[w] = expf(mw[w] - M);
+      L += join[((size_t)w * ROWS_HEADS + row) * (vdim + 2) + vdim + 1] * f[w];
+    }
+    if (splits > 1) {
+      float* dst = partial + (((size_t)t * hq + h) * splits + blockIdx.y) * (vdim + 2);
+      if (lane == 0) { dst[0] = M; dst[1] = L; }
+      for (int d = lane; d < vdim; d += 32) {
+        float sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < ROWS_WARPS; ++w) sum = fmaf(join[((size_t)w * ROWS_HEADS + row) * (vdim + 2) + d], f[w], sum);
+        dst[2 + d] = sum;
+      }
+    } else {
+      const float inv = 1.f / L;
+      for (int d = lane; d < vdim; d += 32) {
+        float sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < ROWS_WARPS; ++w) sum = fmaf(join[((size_t)w * ROWS_HEADS + row) * (vdim + 2) + d], f[w], sum);
+        out[(size_t)t * tail.ldo + (size_t)h * vdim + d] =
+            __float2bfloat16_rn(sum * inv * tail_factor<__nv_bfloat16>(tail, t, h * vdim + d));
+      }
+    }
+  }
+}
+
 size_t tile_smem(int dp, int vp, int share) {
   return sizeof(float) * ((size_t)dp * 33 + 32 * (size_t)vp + (size_t)TILE_T * share * dp + 2 * (size_t)TILE_T * share +
                           (size_t)TILE_T * share * vp);
@@ -754,6 +974,59 @@ PSB_API int psb_attention_biased(const void* q, int dtype, const void* kv, int k
       psb_launch(attention_biased_merge_kernel<T_>, dim3((unsigned)blocks), dim3(32), 0, stream, (const float*)partial,
                  (const float*)sink, (T_*)out, hq, vdim, splits, tail);
     });
+    PSB_LAUNCH_CHECK("attention_biased_merge");
+  }
+  return 0;
+}
+
+// (hq, hkv, dim, vdim) -> 1 if the tensor-core kernel for single tokens takes the shape
+PSB_API int psb_attention_rows_single_supported(int hq, int hkv, int dim, int vdim) {
+  return hq >= 1 && hkv >= 1 && hq % hkv == 0 && dim >= 16 && dim <= 128 && dim % 16 == 0 && vdim >= 8 && vdim <= 128 && vdim % 8 == 0 ? 1 : 0;
+}
+
+// Every token alone (bfloat16), arguments as for psb_attention_biased; no token is skipped.
+// (q, kv, table, table_width, positions, token_item, bias, sink, out, T, hq, hkv, dim, vdim, page_size, window, chunk, reach, scale,
+//  keep_first, partial [T * hq, splits, vdim + 2] float32 or null, splits, gate, ldg, ldo, out_scale, softcap, stream)
+PSB_API int psb_attention_rows_single(const void* q, const void* kv, const void* table, int table_width, const void* positions,
+                                      const void* token_item, const void* bias, const void* sink, void* out, int T, int hq, int hkv,
+                                      int dim, int vdim, int page_size, int window, int chunk, int reach, float scale, int keep_first,
+                                      void* partial, int splits, const void* gate, long long ldg, long long ldo, float out_scale,
+                                      float softcap, cudaStream_t stream) {
+  if (!psb_attention_rows_single_supported(hq, hkv, dim, vdim)) PSB_REFUSE("attention_rows_single: shape not taken");
+  if (splits < 1 || splits > MAX_KEY_SPLITS || (splits > 1 && !partial)) PSB_REFUSE("attention_rows_single: 1 to %d shares of the keys (with their scratch), not %d", MAX_KEY_SPLITS, splits);
+  if (keep_first < 0 || (keep_first > 0 && (window < 1 || chunk > 0))) PSB_REFUSE("attention_rows_single: kept first keys go with a window and no chunk mask");
+  if (T < 0 || page_size < 1 || table_width < 1 || window < 0 || chunk < 0 || (bias && reach < 1)) PSB_REFUSE("attention_rows_single: bad arguments");
+  if (ldo < (long long)hq * vdim || (gate && ldg < (long long)hq * vdim) || softcap < 0.f) PSB_REFUSE("attention_rows_single: bad output or gate rows, or a negative cap");
+  if (((uintptr_t)kv & 15) || ((uintptr_t)q & 3)) PSB_REFUSE("attention_rows_single: cache rows must start on 16 bytes");
+  if (T == 0) return 0;
+  const RowsTail tail{gate, ldg, ldo, out_scale, softcap};
+  const int groups = (hq / hkv + ROWS_HEADS - 1) / ROWS_HEADS;
+  const long long blocks = (long long)T * hkv * groups;
+  if (blocks > 0x7fffffffLL) PSB_REFUSE("attention_rows_single: batch too large");
+  const size_t smem = rows_smem(dim, vdim);
+#define ROWS_CASE(D_, V_)                                                                                                      \
+  do {                                                                                                                         \
+    static PsbPerDevice configured;                                                                                            \
+    if (!configured.get()) {                                                                                                   \
+      if (cudaFuncSetAttribute(attention_rows_single_kernel<D_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize,               \
+                               (int)rows_smem(D_, V_)) != cudaSuccess)                                                         \
+        PSB_REFUSE("attention_rows_single: cannot raise the shared-memory limit");                                             \
+      configured.set();                                                                                                        \
+    }                                                                                                                          \
+    psb_launch(attention_rows_single_kernel<D_, V_>, dim3((unsigned)blocks, (unsigned)splits), dim3(ROWS_WARPS * 32), smem, stream, \
+               (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv, (const int32_t*)table, table_width, (const int32_t*)positions, \
+               (const int32_t*)token_item, (const float*)bias, (const float*)sink, (__nv_bfloat16*)out, hq, hkv, dim, vdim,     \
+               page_size, window, chunk, reach, scale, keep_first, (float*)partial, splits, tail);                             \
+  } while (0)
+  if (dim <= 64 && vdim <= 64) ROWS_CASE(64, 64);
+  else if (dim <= 64) ROWS_CASE(64, 128);
+  else if (vdim <= 64) ROWS_CASE(128, 64);
+  else ROWS_CASE(128, 128);
+#undef ROWS_CASE
+  PSB_LAUNCH_CHECK("attention_rows_single");
+  if (splits > 1) {
+    psb_launch(attention_biased_merge_kernel<__nv_bfloat16>, dim3((unsigned)(T * hq)), dim3(32), 0, stream, (const float*)partial,
+               (const float*)sink, (__nv_bfloat16*)out, hq, vdim, splits, tail);
     PSB_LAUNCH_CHECK("attention_biased_merge");
   }
   return 0;

@@ -390,7 +390,7 @@ attention_prepare_heads_kernel(const HeadsArgs<T> a, TKV* __restrict__ kv) {
 // warps) hold query and key heads, the ones behind them values.  A rotation of halves finds its partner 8 columns times a power
 // of two away, one exchange between two lanes.
 template <typename T, typename TKV, int LPH, int TOK>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(256)
 attention_prepare_heads_vec_kernel(const HeadsArgs<T> a, TKV* __restrict__ kv) {
   pdl_trigger();
   const int heads = a.hq + a.hkv, dim = 8 * LPH;
@@ -506,10 +506,10 @@ attention_prepare_heads_vec_kernel(const HeadsArgs<T> a, TKV* __restrict__ kv) {
 template <typename T, typename TKV, int LPH>
 void launch_heads_vec(const HeadsArgs<T>& a, TKV* kv, cudaStream_t stream) {
   const int lanes = (((a.hq + a.hkv) * LPH + 31) & ~31) + ((a.hkv * (a.vdim / 8) + 31) & ~31);
-  const int threads = lanes < 512 ? lanes : 512;
-  const int tok = a.tokens >= 1024 ? 4 : 1;
+  const int threads = lanes < 256 ? lanes : 256;
+  const int tok = a.tokens >= 512 ? 2 : 1;
   const dim3 grid((a.tokens + tok - 1) / tok, (lanes + threads - 1) / threads);
-  if (tok == 4) psb_launch(attention_prepare_heads_vec_kernel<T, TKV, LPH, 4>, grid, dim3(threads), 0, stream, a, kv);
+  if (tok == 2) psb_launch(attention_prepare_heads_vec_kernel<T, TKV, LPH, 2>, grid, dim3(threads), 0, stream, a, kv);
   else psb_launch(attention_prepare_heads_vec_kernel<T, TKV, LPH, 1>, grid, dim3(threads), 0, stream, a, kv);
 }
 

@@ -897,6 +897,9 @@ BIASED_MMA_MIN_TOKENS = 1
 # every one of them a chain of a thousand keys).  BIASED_BLOCKS_WANTED blocks keep every SM busy; no share below 128 keys.
 BIASED_SPLIT_DECODE = True
 BIASED_BLOCKS_WANTED = 2368
+# ... and of bfloat16 ones whose sizes its tensor-core kernel takes: blocks of (token, key/value head, share of the keys) to aim at
+ROWS_SINGLE = True
+ROWS_BLOCKS_WANTED = 592
 
 
 def biased_attention(qkv: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, ctx, *, num_heads: int, num_kv_heads: int,
@@ -971,6 +974,16 @@ def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, 
             keys = min(keys, win + keep_first)
         if chk:
             keys = min(keys, chk)
+        if (both16 and ROWS_SINGLE and kv.data_ptr() % 16 == 0 and q.data_ptr() % 4 == 0
+                and bool(lib().psb_attention_rows_single_supported(num_heads, num_kv_heads, dim, vdim))):
+            blocks = t * num_kv_heads * -(-(num_heads // num_kv_heads) // 16)
+            splits = max(1, min(16, -(-ROWS_BLOCKS_WANTED // max(blocks, 1)), keys // 64))
+            partial = torch.empty((t, num_heads, splits, vdim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+            check(lib().psb_attention_rows_single(q.data_ptr(), kv.data_ptr(), table.data_ptr(), table.shape[1], positions.data_ptr(),
+                                                  token_item.data_ptr(), _ptr(bias), _ptr(sink), out.data_ptr(), t, num_heads, num_kv_heads,
+                                                  dim, vdim, page_size, win, chk, reach, float(scale), keep_first, _ptr(partial), splits,
+                                                  *tail, _stream()), "attention_rows_single")
+            return out
         splits = max(1, min(16, -(-BIASED_BLOCKS_WANTED // max(t * num_heads, 1)), keys // 128))
         partial = torch.empty((t, num_heads, splits, vdim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
         check(lib().psb_attention_biased(q.data_ptr(), _code(q, "queries"), kv.data_ptr(), _code(kv, "cache entry"),

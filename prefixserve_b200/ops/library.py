@@ -170,6 +170,10 @@ _SIGNATURES: dict[str, list] = {
     # (q, dtype, kv, kv_dtype, table, table_width, positions, token_item, bias, sink, out, T, hq, hkv, dim, vdim, page_size,
     #  window, chunk, reach, scale, item_start, skip_from, stream)
     "psb_attention_biased": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, I, I, P, I, P, L, L, F, F, P],
+    # (q, kv, table, table_width, positions, token_item, bias, sink, out, T, hq, hkv, dim, vdim, page_size, window, chunk, reach, scale,
+    #  keep_first, partial, splits, gate, ldg, ldo, out_scale, softcap, stream)
+    "psb_attention_rows_single": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, P, L, L, F, F, P],
+    "psb_attention_rows_single_supported": [I, I, I, I],
     "psb_attention_biased_tile_tokens": [],
     "psb_attention_biased_tile_supported": [I, I, I, I],
     # (q, kv, table, table_width, positions, item_start, items, T, min_tokens, bias, sink, out, hq, hkv, dim, vdim,
