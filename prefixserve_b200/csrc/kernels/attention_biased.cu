@@ -448,15 +448,6 @@ attention_biased_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
   }
 }
 
-// Prompt portions in bfloat16 on the tensor cores (mma.sync m16n8k16, float32 sums): a block of four warps takes 64
-// consecutive tokens of one request and one query head, a warp 16 of them.  Keys come in blocks of 64 aligned to
-// absolute positions: K as [key][d] and V transposed as [v][key] in shared memory (zeros for keys outside the tile's
-// reach, so nothing of a page that was never written is read).  S = Q K^T stays in the accumulator registers, where
-// scale, bias, masks and the online softmax (started from the sink) are applied in float32; the weights enter the
-// second product as the sum of two bfloat16 numbers (p = hi + lo, two instructions), so they keep 16 bits.
-constexpr int MMA_ROWS = 64, MMA_KEYS = 64;
-constexpr int MMA_BIAS = 2048;  // distances whose bias a block keeps in shared memory
-
 __device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -472,69 +463,70 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16(a - __bfloat162float(ha), b - __bfloat162float(hb));
 }
 
+__device__ __forceinline__ void rows_ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rows_ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void rows_copy16(uint32_t dst, const void* src, bool there) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(there ? 16 : 0) : "memory");
+}
+
+// elements between the rows of a ring: an odd number of 16-byte pieces, so that ldmatrix meets every bank once
+__host__ __device__ __forceinline__ int rows_pitch(int row) { return (row / 8) % 2 ? row : row + 8; }
+// cap * tanh(x / cap) with x = s * scale, as cap - 2 cap / (exp(2 x / cap) + 1): an error of a few units in the last place of the
+// cap, and far out it reaches +-cap.  ``rate`` = 2 log2(e) scale / cap.
+__device__ __forceinline__ float quick_cap(float s, float rate, float cap) { return fmaf(-2.f * cap, __fdividef(1.f, exp2f(s * rate) + 1.f), cap); }
+
+// Prompt portions in bfloat16 on the tensor cores (mma.sync m16n8k16, float32 sums): a block of eight warps takes 128 (token, query
+// head) rows of one request, a warp 16 tokens of one head: 128 consecutive tokens of one head, or 64 of two heads that read the
+// same keys and values.  Keys come in blocks of 64 aligned to absolute positions, whole cache rows (key, then value) brought in
+// with cp.async one block ahead of the arithmetic (zeros for keys outside the tile's reach, so nothing of a page that was never
+// written is read).  S = Q K^T stays in the accumulator registers, where scale, cap, bias, masks and the online softmax (powers of
+// two, started from the sink) are applied in float32; the weights enter the second product as the sum of two bfloat16 numbers
+// (p = hi + lo, two instructions), so they keep 16 bits.  Late tiles, which see the most keys, are started first.
+constexpr int MMA_WARPS = 8, MMA_KEYS = 64;
+constexpr int MMA_BIAS = 2048;  // distances whose bias a block keeps in shared memory, per head
+
+inline size_t mma_smem(int dim, int vdim, bool bias, int heads) {
+  return (size_t)2 * MMA_KEYS * rows_pitch(dim + vdim) * 2 + 32 + (bias ? (size_t)heads * MMA_BIAS * 4 : 0);
+}
+
 template <int D, int V>  // key and value sizes rounded up to 64 or 128
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(MMA_WARPS * 32)
 attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kv,
                             const int32_t* __restrict__ table, int table_width, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ item_start, int items, int min_tokens, const float* __restrict__ bias,
                             const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int hq, int hkv, int dim, int vdim,
-                            int page_size, int window, int chunk, int reach, float scale, int keep_first, const RowsTail tail) {
-  constexpr int KS = D + 8, VS = MMA_KEYS + 8;  // row pitches that keep the fragment loads off each other's banks
-  __shared__ __align__(16) __nv_bfloat16 ks[MMA_KEYS * KS];   // keys [key][d]; first the tile's queries [row][d]
-  __shared__ __align__(16) __nv_bfloat16 vt[V * VS];          // values transposed [v][key]
-  __shared__ float near_bias[MMA_BIAS];                       // the head's bias for the nearest distances
+                            int page_size, int window, int chunk, int reach, float scale, int keep_first, int heads_here, const RowsTail tail) {
+  extern __shared__ __align__(16) unsigned char mma_raw[];
   pdl_wait();
-  int item = -1, t0 = 0;
-  for (int i = 0, left = blockIdx.x; i < items; ++i) {
+  const int tile_tokens = 16 * MMA_WARPS / heads_here;
+  int item = -1, t0 = 0, tiles = 0;
+  for (int i = 0; i < items; ++i) {
+    const int n = item_start[i + 1] - item_start[i];
+    if (n >= min_tokens) tiles += (n + tile_tokens - 1) / tile_tokens;
+  }
+  for (int i = 0, left = tiles - 1 - (int)blockIdx.y; i < items && left >= 0; ++i) {
     const int a = item_start[i], n = item_start[i + 1] - a;
     if (n < min_tokens) continue;
-    const int tiles = (n + MMA_ROWS - 1) / MMA_ROWS;
-    if (left < tiles) { item = i; t0 = a + left * MMA_ROWS; break; }
-    left -= tiles;
+    const int mine = (n + tile_tokens - 1) / tile_tokens;
+    if (left < mine) { item = i; t0 = a + left * tile_tokens; break; }
+    left -= mine;
   }
   if (item < 0) return;
-  const int h = blockIdx.y, g = h / (hq / hkv);
-  const int nt = min(MMA_ROWS, item_start[item + 1] - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-  const int rw = dim + vdim;
+  const int warps_a_head = MMA_WARPS / heads_here;
+  const int h0 = blockIdx.x * heads_here, which = warp / warps_a_head, h = h0 + which, g = h / (hq / hkv);
+  const int row0 = (warp - which * warps_a_head) * 16;  // this warp's first token of the tile
+  const int nt = min(tile_tokens, item_start[item + 1] - t0);
+  const int rw = dim + vdim, pitch = rows_pitch(rw), pieces = rw / 8;
   const size_t head_stride = (size_t)page_size * rw, page_elems = (size_t)hkv * head_stride;
   const int32_t* pages = table + (size_t)item * table_width;
   const int p_first = positions[t0], p_last = p_first + nt - 1;
-
-  // the tile's queries through shared memory into fragments
-  for (int i = threadIdx.x; i < MMA_ROWS * (D / 8); i += blockDim.x) {
-    const int r = i / (D / 8), c = (i - r * (D / 8)) * 8;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < nt && c < dim) v = *reinterpret_cast<const uint4*>(q + ((size_t)(t0 + r) * hq + h) * dim + c);
-    *reinterpret_cast<uint4*>(&ks[r * KS + c]) = v;
-  }
-  __syncthreads();
-  uint32_t qf[D / 16][4];
-#pragma unroll
-  for (int kk = 0; kk < D / 16; ++kk) {
-    qf[kk][0] = *reinterpret_cast<const uint32_t*>(&ks[(warp * 16 + gid) * KS + kk * 16 + 2 * tig]);
-    qf[kk][1] = *reinterpret_cast<const uint32_t*>(&ks[(warp * 16 + gid + 8) * KS + kk * 16 + 2 * tig]);
-    qf[kk][2] = *reinterpret_cast<const uint32_t*>(&ks[(warp * 16 + gid) * KS + kk * 16 + 2 * tig + 8]);
-    qf[kk][3] = *reinterpret_cast<const uint32_t*>(&ks[(warp * 16 + gid + 8) * KS + kk * 16 + 2 * tig + 8]);
-  }
-  // this thread's two rows: positions, lowest visible keys, running maximum and its share of the running sum
-  int pos[2], low[2];
-  float m[2], l[2];
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    pos[r] = p_first + warp * 16 + gid + 8 * r;
-    low[r] = (window > 0 && pos[r] - window + 1 > 0) ? pos[r] - window + 1 : 0;
-    if (chunk > 0) low[r] = max(low[r], (pos[r] / chunk) * chunk);
-    if (keep_first > 0 && low[r] <= keep_first) low[r] = 0;
-    m[r] = sink ? sink[h] : -FLT_MAX;
-    l[r] = (sink && tig == 0) ? 1.f : 0.f;
-  }
-  float o[V / 8][4];
-#pragma unroll
-  for (int i = 0; i < V / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  const float* brow = bias ? bias + (size_t)h * reach : nullptr;
-  if (brow)
-    for (int i = threadIdx.x; i < min(reach, MMA_BIAS); i += 128) near_bias[i] = brow[i];  // visible after the loop's first barrier
+  const uint32_t ring = (uint32_t)__cvta_generic_to_shared(mma_raw);
+  float* near_bias = reinterpret_cast<float*>(mma_raw + (size_t)2 * MMA_KEYS * pitch * 2 + 32);  // the heads' bias for the nearest distances
 
   int lo_tile = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
   if (chunk > 0) lo_tile = max(lo_tile, (p_first / chunk) * chunk);
@@ -544,90 +536,122 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     if (lo_tile <= keep_first) lo_tile = 0;
     else kept_blocks = (keep_first + MMA_KEYS - 1) / MMA_KEYS;
   }
-  for (int blk = 0;; ++blk) {
-    const bool kept = blk < kept_blocks;
-    const int base = kept ? MMA_KEYS * blk : (lo_tile & ~(MMA_KEYS - 1)) + MMA_KEYS * (blk - kept_blocks);
-    if (base > p_last) break;
-    __syncthreads();  // everybody has its query fragments (first round) or is done with the last block
-    // every thread asks for all its pieces of the block (page ids first, then the rows) before it stores any
-    constexpr int KPIECES = MMA_KEYS * (D / 8) / 128, VPIECES = MMA_KEYS * (V / 8) / 128;
-    uint4 kreg[KPIECES], vreg[VPIECES];
+  const int blocks = kept_blocks + p_last / MMA_KEYS - lo_tile / MMA_KEYS + 1;
+  auto base_of = [&](int blk) { return MMA_KEYS * (blk < kept_blocks ? blk : lo_tile / MMA_KEYS + blk - kept_blocks); };
+  auto fetch = [&](int blk) {
+    if (blk < blocks) {
+      const int base = base_of(blk) + warp * (MMA_KEYS / MMA_WARPS);
+      long long off = -1;  // lane r: where this warp's row r of the block lies
+      if (lane < MMA_KEYS / MMA_WARPS) {
+        const int key = base + lane;
+        if (blk < kept_blocks ? key < keep_first : (key >= lo_tile && key <= p_last))
+          off = (long long)((size_t)pages[key / page_size] * page_elems + (size_t)g * head_stride + (size_t)(key % page_size) * rw);
+      }
+      const uint32_t dst = ring + (uint32_t)(((blk & 1) * MMA_KEYS + warp * (MMA_KEYS / MMA_WARPS)) * pitch * 2);
 #pragma unroll
-    for (int u = 0; u < KPIECES; ++u) {
-      const int i = threadIdx.x + u * 128;
-      const int j = i / (D / 8), c = (i - j * (D / 8)) * 8;
-      const int key = base + j;
-      kreg[u] = make_uint4(0, 0, 0, 0);
-      if ((kept ? key < keep_first : (key >= lo_tile && key <= p_last)) && c < dim)
-        kreg[u] = *reinterpret_cast<const uint4*>(kv + (size_t)pages[key / page_size] * page_elems + (size_t)g * head_stride +
-                                                  (size_t)(key % page_size) * rw + c);
-    }
-#pragma unroll
-    for (int u = 0; u < VPIECES; ++u) {
-      const int i = threadIdx.x + u * 128;
-      const int j = i % MMA_KEYS, c = (i / MMA_KEYS) * 8;  // neighbouring lanes: neighbouring keys, the same eight value channels
-      const int key = base + j;
-      vreg[u] = make_uint4(0, 0, 0, 0);
-      if ((kept ? key < keep_first : (key >= lo_tile && key <= p_last)) && c < vdim)
-        vreg[u] = *reinterpret_cast<const uint4*>(kv + (size_t)pages[key / page_size] * page_elems + (size_t)g * head_stride +
-                                                  (size_t)(key % page_size) * rw + dim + c);
-    }
-#pragma unroll
-    for (int u = 0; u < KPIECES; ++u) {
-      const int i = threadIdx.x + u * 128;
-      const int j = i / (D / 8), c = (i - j * (D / 8)) * 8;
-      *reinterpret_cast<uint4*>(&ks[j * KS + c]) = kreg[u];
-    }
-#pragma unroll
-    for (int u = 0; u < VPIECES; ++u) {
-      const int i = threadIdx.x + u * 128;
-      const int j = i % MMA_KEYS, c = (i / MMA_KEYS) * 8;
-      const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&vreg[u]);
-#pragma unroll
-      for (int k = 0; k < 8; ++k) vt[(c + k) * VS + j] = e[k];
-    }
-    __syncthreads();
-    if (warp * 16 >= nt || base > p_first + warp * 16 + 15) continue;  // no rows, or all of them before the block (uniform in the warp)
-    // (a kept block lies before every row of a tile that has any: then every row's window starts beyond keep_first)
-    float sc[MMA_KEYS / 8][4];
-#pragma unroll
-    for (int n = 0; n < MMA_KEYS / 8; ++n) {
-      sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
-#pragma unroll
-      for (int kk = 0; kk < D / 16; ++kk) {
-        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(&ks[(n * 8 + gid) * KS + kk * 16 + 2 * tig]);
-        const uint32_t b1 = *reinterpret_cast<const uint32_t*>(&ks[(n * 8 + gid) * KS + kk * 16 + 2 * tig + 8]);
-        mma_16816(sc[n], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
+      for (int r = 0; r < MMA_KEYS / MMA_WARPS; ++r) {
+        const long long at = __shfl_sync(0xffffffffu, off, r);
+        for (int c = lane; c < pieces; c += 32) rows_copy16(dst + (uint32_t)(r * pitch + c * 8) * 2, kv + (at < 0 ? 0 : at) + c * 8, at >= 0);
       }
     }
-    float top[2] = {-FLT_MAX, -FLT_MAX};
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0);
+
+  uint32_t qf[D / 16][4];
+#pragma unroll
+  for (int kk = 0; kk < D / 16; ++kk)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = row0 + gid + 8 * (e & 1), c = kk * 16 + 2 * tig + 8 * (e >> 1);
+      qf[kk][e] = row < nt && c < dim ? *reinterpret_cast<const uint32_t*>(q + ((size_t)(t0 + row) * hq + h) * dim + c) : 0u;
+    }
+  // this thread's two rows: positions, lowest visible keys, running maximum and its share of the running sum
+  int pos[2], low[2];
+  float m[2], l[2];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    pos[r] = p_first + row0 + gid + 8 * r;
+    low[r] = (window > 0 && pos[r] - window + 1 > 0) ? pos[r] - window + 1 : 0;
+    if (chunk > 0) low[r] = max(low[r], (pos[r] / chunk) * chunk);
+    if (keep_first > 0 && low[r] <= keep_first) low[r] = 0;
+    m[r] = sink ? sink[h] * PSB_LOG2E : -FLT_MAX;
+    l[r] = (sink && tig == 0) ? 1.f : 0.f;
+  }
+  // what the warp's rows see as a whole: every key of [all_from, all_to], none below none_below (the lowest is the first row's)
+  const int w_first = p_first + row0, w_last = w_first + 15;
+  const int none_below = __shfl_sync(0xffffffffu, low[0], 0), all_from = __shfl_sync(0xffffffffu, low[1], 31), all_to = w_first;
+  float o[V / 8][4];
+#pragma unroll
+  for (int i = 0; i < V / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  if (bias)
+    for (int i = threadIdx.x; i < heads_here * MMA_BIAS; i += MMA_WARPS * 32) {
+      const int d = i % MMA_BIAS;
+      near_bias[i] = d < reach ? bias[(size_t)(h0 + i / MMA_BIAS) * reach + d] * PSB_LOG2E : 0.f;  // visible after the loop's first barrier
+    }
+  const float* brow = bias ? bias + (size_t)h * reach : nullptr;
+  const float factor = scale * PSB_LOG2E, cap = tail.softcap * PSB_LOG2E, rate = tail.softcap > 0.f ? 2.f * PSB_LOG2E * scale / tail.softcap : 0.f;
+  const int lrow = lane & 7, lmat = lane >> 3;
+
+  for (int blk = 0; blk < blocks; ++blk) {
+    const bool kept = blk < kept_blocks;
+    const int base = base_of(blk);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // this block has landed for everybody, and everybody is done with the other buffer
+    fetch(blk + 1);
+    // no rows, or all of them before the block or (without kept keys) beyond what they see (uniform in the warp)
+    if (row0 >= nt || base > w_last || (keep_first == 0 && base + MMA_KEYS - 1 < none_below)) continue;
+    const uint32_t src = ring + (uint32_t)((blk & 1) * MMA_KEYS * pitch * 2);
+    float sc[MMA_KEYS / 8][4];
+#pragma unroll
+    for (int n = 0; n < MMA_KEYS / 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      if (kk * 16 >= dim) break;  // (keys in an odd number of eights: the last step meets value channels with zeros of q)
+#pragma unroll
+      for (int n = 0; n < MMA_KEYS / 8; n += 2) {
+        uint32_t b[4];
+        rows_ldmatrix4(b, src + (uint32_t)((n * 8 + (lmat >> 1) * 8 + lrow) * pitch + kk * 16 + (lmat & 1) * 8) * 2);
+        mma_16816(sc[n], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[0], b[1]);
+        mma_16816(sc[n + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[2], b[3]);
+      }
+    }
     if (tail.softcap > 0.f) {
-      // cap * tanh(s * scale / cap) / scale as cap / scale * (1 - 2 / (exp(2 s scale / cap) + 1)): an error of a few units in
-      // the last place of the cap, far out it reaches +-cap (the scale itself is applied below)
-      const float far = tail.softcap / scale, rate = 2.f * PSB_LOG2E / far;
 #pragma unroll
       for (int n = 0; n < MMA_KEYS / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[n][e] = fmaf(-2.f * far, __fdividef(1.f, exp2f(sc[n][e] * rate) + 1.f), far);
+        for (int e = 0; e < 4; ++e) sc[n][e] = quick_cap(sc[n][e], rate, cap);
+    } else {
+#pragma unroll
+      for (int n = 0; n < MMA_KEYS / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[n][e] *= factor;
     }
+    if (brow) {
+#pragma unroll
+      for (int n = 0; n < MMA_KEYS / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int far = max(0, min(pos[e >> 1] - (base + n * 8 + 2 * tig + (e & 1)), reach - 1));
+          sc[n][e] += far < MMA_BIAS ? near_bias[which * MMA_BIAS + far] : brow[far] * PSB_LOG2E;
+        }
+    }
+    if (kept || base < all_from || base + MMA_KEYS - 1 > all_to) {
+      // (without kept blocks of their own the kept keys lie inside the ordinary blocks: a later row of the tile may see them
+      // although its window starts beyond them; a kept block lies before every row of a tile that has any)
+#pragma unroll
+      for (int n = 0; n < MMA_KEYS / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = e >> 1, key = base + n * 8 + 2 * tig + (e & 1);
+          if (!(kept ? key < keep_first : (key <= pos[r] && (key >= low[r] || (kept_blocks == 0 && key < keep_first))))) sc[n][e] = -INFINITY;
+        }
+    }
+    float top[2] = {-FLT_MAX, -FLT_MAX};
 #pragma unroll
     for (int n = 0; n < MMA_KEYS / 8; ++n) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = e >> 1, key = base + n * 8 + 2 * tig + (e & 1);
-        float v = -INFINITY;
-        // (without kept blocks of their own the kept keys lie inside the ordinary blocks: a later row of the tile may
-        // see them although its window starts beyond them)
-        if (kept ? key < keep_first : (key <= pos[r] && (key >= low[r] || (kept_blocks == 0 && key < keep_first)))) {
-          v = sc[n][e] * scale;
-          if (brow) {
-            const int far = min(pos[r] - key, reach - 1);
-            v += far < MMA_BIAS ? near_bias[far] : brow[far];
-          }
-        }
-        sc[n][e] = v;
-        top[r] = fmaxf(top[r], v);
-      }
+      top[0] = fmaxf(top[0], fmaxf(sc[n][0], sc[n][1]));
+      top[1] = fmaxf(top[1], fmaxf(sc[n][2], sc[n][3]));
     }
     float alpha[2];
 #pragma unroll
@@ -635,18 +659,9 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
       top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
       const float m_new = fmaxf(m[r], top[r]);
-      alpha[r] = expf(m[r] - m_new);
+      alpha[r] = exp2f(m[r] - m_new);
       m[r] = m_new;
       l[r] *= alpha[r];
-    }
-#pragma unroll
-    for (int n = 0; n < MMA_KEYS / 8; ++n) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float pv = expf(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
-        sc[n][e] = pv;
-        l[e >> 1] += pv;
-      }
     }
 #pragma unroll
     for (int i = 0; i < V / 8; ++i) {
@@ -655,17 +670,27 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     }
 #pragma unroll
     for (int kk = 0; kk < MMA_KEYS / 16; ++kk) {
+#pragma unroll
+      for (int n = 2 * kk; n < 2 * kk + 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[n][e] = exp2f(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
+          l[e >> 1] += sc[n][e];
+        }
       uint32_t hi[4], lo[4];
       split_bf16(sc[2 * kk][0], sc[2 * kk][1], hi[0], lo[0]);
       split_bf16(sc[2 * kk][2], sc[2 * kk][3], hi[1], lo[1]);
       split_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1], hi[2], lo[2]);
       split_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3], hi[3], lo[3]);
 #pragma unroll
-      for (int nv = 0; nv < V / 8; ++nv) {
-        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(&vt[(nv * 8 + gid) * VS + kk * 16 + 2 * tig]);
-        const uint32_t b1 = *reinterpret_cast<const uint32_t*>(&vt[(nv * 8 + gid) * VS + kk * 16 + 2 * tig + 8]);
-        mma_16816(o[nv], hi[0], hi[1], hi[2], hi[3], b0, b1);
-        mma_16816(o[nv], lo[0], lo[1], lo[2], lo[3], b0, b1);
+      for (int nv = 0; nv < V / 8; nv += 2) {
+        if (nv * 8 >= vdim) break;
+        uint32_t b[4];  // (values in an odd number of eights: the last columns read 16 bytes beyond the row, and nobody stores them)
+        rows_ldmatrix4_trans(b, src + (uint32_t)((kk * 16 + (lmat & 1) * 8 + lrow) * pitch + dim + nv * 8 + (lmat >> 1) * 8) * 2);
+        mma_16816(o[nv], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+        mma_16816(o[nv + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+        mma_16816(o[nv], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+        mma_16816(o[nv + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
       }
     }
   }
@@ -677,7 +702,7 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
-    const int row = warp * 16 + gid + 8 * r;
+    const int row = row0 + gid + 8 * r;
     if (row >= nt) continue;
     const float inv = 1.f / l[r];
     __nv_bfloat16* orow = out + (size_t)(t0 + row) * tail.ldo + (size_t)h * vdim;
@@ -700,18 +725,6 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 // above joins them.
 constexpr int ROWS_WARPS = 4, ROWS_RUN = 16, ROWS_HEADS = 16, ROWS_STAGES = 3;
 
-__device__ __forceinline__ void rows_ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void rows_ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void rows_copy16(uint32_t dst, const void* src, bool there) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(there ? 16 : 0) : "memory");
-}
-
-// elements between the rows of a ring: an odd number of 16-byte pieces, so that ldmatrix meets every bank once
-__host__ __device__ __forceinline__ int rows_pitch(int row) { return (row / 8) % 2 ? row : row + 8; }
 inline size_t rows_smem(int dim, int vdim) {
   const size_t ring = (size_t)ROWS_WARPS * ROWS_STAGES * ROWS_RUN * rows_pitch(dim + vdim) * 2 + 32;
   const size_t join = (size_t)ROWS_WARPS * ROWS_HEADS * (vdim + 2) * 4;
@@ -785,6 +798,7 @@ attention_rows_single_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 #pragma unroll
   for (int i = 0; i < V / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   const int lrow = lane & 7, lmat = lane >> 3;
+  const float rate = tail.softcap > 0.f ? 2.f * PSB_LOG2E * scale / tail.softcap : 0.f;
   int stage = 0;
   for (int run = mine; run < runs; run += step) {
     asm volatile("cp.async.wait_group %0;" ::"n"(ROWS_STAGES - 2) : "memory");
@@ -809,8 +823,8 @@ attention_rows_single_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = e >> 1, key = base + n * 8 + 2 * tig + (e & 1);
-        float v = sc[n][e] * scale;
-        if (tail.softcap > 0.f) v = tail.softcap * tanhf(v / tail.softcap);
+        if (r == 1 && heads <= 8) break;  // no heads in the upper rows (the same for the whole block)
+        float v = tail.softcap > 0.f ? quick_cap(sc[n][e], rate, tail.softcap) : sc[n][e] * scale;
         if (bias && gid + 8 * r < heads) v += bias[(size_t)(h0 + gid + 8 * r) * reach + max(0, min(p - key, reach - 1))];
         if (!(kept ? key < keep_first : (key >= lo && key <= p))) v = -INFINITY;
         sc[n][e] = v;
@@ -818,6 +832,7 @@ attention_rows_single_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
       }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
+      if (r == 1 && heads <= 8) break;
       top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
       top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
       const float m_new = fmaxf(m[r], top[r]), alpha = expf(m[r] - m_new);
@@ -830,6 +845,7 @@ attention_rows_single_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
+        if (e >> 1 == 1 && heads <= 8) { sc[n][e] = 0.f; continue; }
         sc[n][e] = expf(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
         l[e >> 1] += sc[n][e];
       }
@@ -981,7 +997,7 @@ PSB_API int psb_attention_biased(const void* q, int dtype, const void* kv, int k
 
 // (hq, hkv, dim, vdim) -> 1 if the tensor-core kernel for single tokens takes the shape
 PSB_API int psb_attention_rows_single_supported(int hq, int hkv, int dim, int vdim) {
-  return hq >= 1 && hkv >= 1 && hq % hkv == 0 && dim >= 16 && dim <= 128 && dim % 16 == 0 && vdim >= 8 && vdim <= 128 && vdim % 8 == 0 ? 1 : 0;
+  return hq >= 1 && hkv >= 1 && hq % hkv == 0 && dim >= 8 && dim <= 128 && dim % 8 == 0 && vdim >= 8 && vdim <= 128 && vdim % 8 == 0 ? 1 : 0;
 }
 
 // Every token alone (bfloat16), arguments as for psb_attention_biased; no token is skipped.
@@ -1038,7 +1054,7 @@ PSB_API int psb_attention_biased_mma_supported(int hq, int hkv, int dim, int vdi
 }
 
 // The tensor-core kernel over every portion of at least ``min_tokens`` tokens (bfloat16; grid sized by an upper bound on
-// the 64-token tiles).  Other tokens are left untouched.
+// the tiles).  Other tokens are left untouched.
 // (q, kv, table, table_width, positions, item_start, items, T, min_tokens, bias, sink, out, hq, hkv, dim, vdim,
 //  page_size, window, chunk, reach, scale, keep_first, gate, ldg, ldo, out_scale, softcap, stream)
 PSB_API int psb_attention_biased_mma(const void* q, const void* kv, const void* table, int table_width, const void* positions,
@@ -1048,19 +1064,31 @@ PSB_API int psb_attention_biased_mma(const void* q, const void* kv, const void* 
                                      float softcap, cudaStream_t stream) {
   if (ldo < (long long)hq * vdim || ldo % 2 || ((uintptr_t)out & 3) || (gate && ldg < (long long)hq * vdim) || softcap < 0.f)
     PSB_REFUSE("attention_biased_mma: bad output or gate rows, or a negative cap");
-  if (softcap > 0.f && scale == 0.f) PSB_REFUSE("attention_biased_mma: a cap needs a scale that is not zero");
   const RowsTail tail{gate, ldg, ldo, out_scale, softcap};
   if (!psb_attention_biased_mma_supported(hq, hkv, dim, vdim)) PSB_REFUSE("attention_biased_mma: shape not taken");
   if (keep_first < 0 || (keep_first > 0 && (window < 1 || chunk > 0))) PSB_REFUSE("attention_biased_mma: kept first keys go with a window and no chunk mask");
   if (page_size < 1 || table_width < 1 || window < 0 || chunk < 0 || (bias && reach < 1)) PSB_REFUSE("attention_biased_mma: bad arguments");
   if ((((uintptr_t)q | (uintptr_t)kv) & 15) || hq > 65535) PSB_REFUSE("attention_biased_mma: operands must be 16-byte aligned");
   if (items < 1 || T < 1 || min_tokens < 1) return 0;
-  const dim3 grid((T + MMA_ROWS - 1) / MMA_ROWS + items, hq), block(128);
+  // two heads that read the same keys and values share a block (64 tokens each) where there are such heads
+  const int heads_here = (hq / hkv) % 2 == 0 ? 2 : 1, tile_tokens = 16 * MMA_WARPS / heads_here;
+  const dim3 grid(hq / heads_here, (T + tile_tokens - 1) / tile_tokens + items);
+  if (grid.y > 65535) PSB_REFUSE("attention_biased_mma: %d tokens are too many for one launch", T);
+  const size_t smem = mma_smem(dim, vdim, bias != nullptr, heads_here);
 #define MMA_CASE(D_, V_)                                                                                                       \
-  psb_launch(attention_biased_mma_kernel<D_, V_>, grid, block, 0, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv,    \
-             (const int32_t*)table, table_width, (const int32_t*)positions, (const int32_t*)item_start, items, min_tokens,     \
-             (const float*)bias, (const float*)sink, (__nv_bfloat16*)out, hq, hkv, dim, vdim, page_size, window, chunk, reach, \
-             scale, keep_first, tail)
+  do {                                                                                                                         \
+    static PsbPerDevice configured;                                                                                            \
+    if (!configured.get()) {                                                                                                   \
+      if (cudaFuncSetAttribute(attention_biased_mma_kernel<D_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize,                \
+                               (int)mma_smem(D_, V_, true, 2)) != cudaSuccess)                                                 \
+        PSB_REFUSE("attention_biased_mma: cannot raise the shared-memory limit");                                              \
+      configured.set();                                                                                                        \
+    }                                                                                                                          \
+    psb_launch(attention_biased_mma_kernel<D_, V_>, grid, dim3(MMA_WARPS * 32), smem, stream, (const __nv_bfloat16*)q,          \
+               (const __nv_bfloat16*)kv, (const int32_t*)table, table_width, (const int32_t*)positions,                        \
+               (const int32_t*)item_start, items, min_tokens, (const float*)bias, (const float*)sink, (__nv_bfloat16*)out, hq,  \
+               hkv, dim, vdim, page_size, window, chunk, reach, scale, keep_first, heads_here, tail);                          \
+  } while (0)
   if (dim <= 64 && vdim <= 64) MMA_CASE(64, 64);
   else if (dim <= 64) MMA_CASE(64, 128);
   else if (vdim <= 64) MMA_CASE(128, 64);
