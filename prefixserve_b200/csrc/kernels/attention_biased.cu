@@ -483,18 +483,19 @@ __device__ __forceinline__ float quick_cap(float s, float rate, float cap) { ret
 // head) rows of one request, a warp 16 tokens of one head: 128 consecutive tokens of one head, or 64 of two heads that read the
 // same keys and values.  Keys come in blocks of 64 aligned to absolute positions, whole cache rows (key, then value) brought in
 // with cp.async one block ahead of the arithmetic (zeros for keys outside the tile's reach, so nothing of a page that was never
-// written is read).  S = Q K^T stays in the accumulator registers, where scale, cap, bias, masks and the online softmax (powers of
+// written is read) and worked on 32 at a time; the queries stay in shared memory, so that two blocks fit an SM.  S = Q K^T stays in the accumulator registers, where scale, cap, bias, masks and the online softmax (powers of
 // two, started from the sink) are applied in float32; the weights enter the second product as the sum of two bfloat16 numbers
-// (p = hi + lo, two instructions), so they keep 16 bits.  Late tiles, which see the most keys, are started first.
-constexpr int MMA_WARPS = 8, MMA_KEYS = 64;
-constexpr int MMA_BIAS = 2048;  // distances whose bias a block keeps in shared memory, per head
+// (p = hi + lo, two instructions), so they keep 16 bits.  Late tiles (of a sequence or of its chunks), which see
+// the most keys, are started first.
+constexpr int MMA_WARPS = 8, MMA_KEYS = 64, MMA_PART = 32;
+constexpr int MMA_BIAS = 1024;  // distances whose bias a block keeps in shared memory, per head
 
 inline size_t mma_smem(int dim, int vdim, bool bias, int heads) {
-  return (size_t)2 * MMA_KEYS * rows_pitch(dim + vdim) * 2 + 32 + (bias ? (size_t)heads * MMA_BIAS * 4 : 0);
+  return (size_t)2 * MMA_KEYS * rows_pitch(dim + vdim) * 2 + 32 + (size_t)16 * MMA_WARPS * rows_pitch((dim + 15) / 16 * 16) * 2 + (bias ? (size_t)heads * MMA_BIAS * 4 : 0);
 }
 
 template <int D, int V>  // key and value sizes rounded up to 64 or 128
-__global__ void __launch_bounds__(MMA_WARPS * 32)
+__global__ void __launch_bounds__(MMA_WARPS * 32, 2)
 attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kv,
                             const int32_t* __restrict__ table, int table_width, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ item_start, int items, int min_tokens, const float* __restrict__ bias,
@@ -508,7 +509,13 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const int n = item_start[i + 1] - item_start[i];
     if (n >= min_tokens) tiles += (n + tile_tokens - 1) / tile_tokens;
   }
-  for (int i = 0, left = tiles - 1 - (int)blockIdx.y; i < items && left >= 0; ++i) {
+  int at = tiles - 1 - (int)blockIdx.y;
+  if (chunk >= 2 * tile_tokens && items == 1) {  // (the launch has blocks for this): the late tiles of every chunk, then the ones before them
+    const int per = chunk / tile_tokens, chunks = (tiles + per - 1) / per, round = (int)blockIdx.y / chunks;
+    at = ((int)blockIdx.y - round * chunks) * per + per - 1 - round;
+    if (round >= per || at >= tiles) return;
+  }
+  for (int i = 0, left = at; i < items && left >= 0; ++i) {
     const int a = item_start[i], n = item_start[i + 1] - a;
     if (n < min_tokens) continue;
     const int mine = (n + tile_tokens - 1) / tile_tokens;
@@ -526,7 +533,9 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int32_t* pages = table + (size_t)item * table_width;
   const int p_first = positions[t0], p_last = p_first + nt - 1;
   const uint32_t ring = (uint32_t)__cvta_generic_to_shared(mma_raw);
-  float* near_bias = reinterpret_cast<float*>(mma_raw + (size_t)2 * MMA_KEYS * pitch * 2 + 32);  // the heads' bias for the nearest distances
+  const int q_width = (dim + 15) / 16 * 16, q_pitch = rows_pitch(q_width);
+  unsigned char* q_raw = mma_raw + (size_t)2 * MMA_KEYS * pitch * 2 + 32;  // the warps' queries, 16 rows each
+  float* near_bias = reinterpret_cast<float*>(q_raw + (size_t)16 * MMA_WARPS * q_pitch * 2);  // the heads' bias for the nearest distances
 
   int lo_tile = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
   if (chunk > 0) lo_tile = max(lo_tile, (p_first / chunk) * chunk);
@@ -558,14 +567,14 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   };
   fetch(0);
 
-  uint32_t qf[D / 16][4];
-#pragma unroll
-  for (int kk = 0; kk < D / 16; ++kk)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int row = row0 + gid + 8 * (e & 1), c = kk * 16 + 2 * tig + 8 * (e >> 1);
-      qf[kk][e] = row < nt && c < dim ? *reinterpret_cast<const uint32_t*>(q + ((size_t)(t0 + row) * hq + h) * dim + c) : 0u;
-    }
+  // a warp brings in its own queries and is the only one to read them (rows beyond the portion and columns beyond dim are zeros)
+  for (int i = lane; i < 16 * (q_width / 8); i += 32) {
+    const int r = i / (q_width / 8), c = (i - r * (q_width / 8)) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (row0 + r < nt && c < dim) v = *reinterpret_cast<const uint4*>(q + ((size_t)(t0 + row0 + r) * hq + h) * dim + c);
+    *reinterpret_cast<uint4*>(q_raw + (size_t)((warp * 16 + r) * q_pitch + c) * 2) = v;
+  }
+  __syncwarp();
   // this thread's two rows: positions, lowest visible keys, running maximum and its share of the running sum
   int pos[2], low[2];
   float m[2], l[2];
@@ -592,6 +601,7 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const float* brow = bias ? bias + (size_t)h * reach : nullptr;
   const float factor = scale * PSB_LOG2E, cap = tail.softcap * PSB_LOG2E, rate = tail.softcap > 0.f ? 2.f * PSB_LOG2E * scale / tail.softcap : 0.f;
   const int lrow = lane & 7, lmat = lane >> 3;
+  const uint32_t q_at = (uint32_t)__cvta_generic_to_shared(q_raw) + (uint32_t)((warp * 16 + (lmat & 1) * 8 + lrow) * q_pitch + (lmat >> 1) * 8) * 2;
 
   for (int blk = 0; blk < blocks; ++blk) {
     const bool kept = blk < kept_blocks;
@@ -601,96 +611,106 @@ attention_biased_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     fetch(blk + 1);
     // no rows, or all of them before the block or (without kept keys) beyond what they see (uniform in the warp)
     if (row0 >= nt || base > w_last || (keep_first == 0 && base + MMA_KEYS - 1 < none_below)) continue;
-    const uint32_t src = ring + (uint32_t)((blk & 1) * MMA_KEYS * pitch * 2);
-    float sc[MMA_KEYS / 8][4];
+#pragma unroll 1
+    for (int part = 0; part < MMA_KEYS; part += MMA_PART) {
+      const int key0 = base + part;
+      if (key0 > w_last || (keep_first == 0 && key0 + MMA_PART - 1 < none_below)) continue;
+      const uint32_t src = ring + (uint32_t)(((blk & 1) * MMA_KEYS + part) * pitch * 2);
+      float sc[MMA_PART / 8][4];
 #pragma unroll
-    for (int n = 0; n < MMA_KEYS / 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+      for (int n = 0; n < MMA_PART / 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
 #pragma unroll
-    for (int kk = 0; kk < D / 16; ++kk) {
-      if (kk * 16 >= dim) break;  // (keys in an odd number of eights: the last step meets value channels with zeros of q)
+      for (int kk = 0; kk < D / 16; ++kk) {
+        if (kk * 16 >= dim) break;  // (keys in an odd number of eights: the last step meets value channels with zeros of q)
+        uint32_t a[4];
+        rows_ldmatrix4(a, q_at + (uint32_t)(kk * 32));
 #pragma unroll
-      for (int n = 0; n < MMA_KEYS / 8; n += 2) {
-        uint32_t b[4];
-        rows_ldmatrix4(b, src + (uint32_t)((n * 8 + (lmat >> 1) * 8 + lrow) * pitch + kk * 16 + (lmat & 1) * 8) * 2);
-        mma_16816(sc[n], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[0], b[1]);
-        mma_16816(sc[n + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b[2], b[3]);
+        for (int n = 0; n < MMA_PART / 8; n += 2) {
+          uint32_t b[4];
+          rows_ldmatrix4(b, src + (uint32_t)((n * 8 + (lmat >> 1) * 8 + lrow) * pitch + kk * 16 + (lmat & 1) * 8) * 2);
+          mma_16816(sc[n], a[0], a[1], a[2], a[3], b[0], b[1]);
+          mma_16816(sc[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        }
       }
-    }
-    if (tail.softcap > 0.f) {
+      if (tail.softcap > 0.f) {
 #pragma unroll
-      for (int n = 0; n < MMA_KEYS / 8; ++n)
+        for (int n = 0; n < MMA_PART / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[n][e] = quick_cap(sc[n][e], rate, cap);
-    } else {
+          for (int e = 0; e < 4; ++e) sc[n][e] = quick_cap(sc[n][e], rate, cap);
+      } else {
 #pragma unroll
-      for (int n = 0; n < MMA_KEYS / 8; ++n)
+        for (int n = 0; n < MMA_PART / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[n][e] *= factor;
-    }
-    if (brow) {
+          for (int e = 0; e < 4; ++e) sc[n][e] *= factor;
+      }
+      if (brow) {
 #pragma unroll
-      for (int n = 0; n < MMA_KEYS / 8; ++n)
+        for (int n = 0; n < MMA_PART / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int far = max(0, min(pos[e >> 1] - (base + n * 8 + 2 * tig + (e & 1)), reach - 1));
-          sc[n][e] += far < MMA_BIAS ? near_bias[which * MMA_BIAS + far] : brow[far] * PSB_LOG2E;
+          for (int e = 0; e < 4; ++e) {
+            const int far = max(0, min(pos[e >> 1] - (key0 + n * 8 + 2 * tig + (e & 1)), reach - 1));
+            sc[n][e] += far < MMA_BIAS ? near_bias[which * MMA_BIAS + far] : brow[far] * PSB_LOG2E;
+          }
+      }
+      if (kept || key0 < all_from || key0 + MMA_PART - 1 > all_to) {
+        // (without kept blocks of their own the kept keys lie inside the ordinary blocks: a later row of the tile may see them
+        // although its window starts beyond them; a kept block lies before every row of a tile that has any)
+#pragma unroll
+        for (int n = 0; n < MMA_PART / 8; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int r = e >> 1, key = key0 + n * 8 + 2 * tig + (e & 1);
+            if (!(kept ? key < keep_first : (key <= pos[r] && (key >= low[r] || (kept_blocks == 0 && key < keep_first))))) sc[n][e] = -INFINITY;
+          }
+      }
+      float top[2] = {m[0], m[1]};
+#pragma unroll
+      for (int n = 0; n < MMA_PART / 8; ++n) {
+        top[0] = fmaxf(top[0], fmaxf(sc[n][0], sc[n][1]));
+        top[1] = fmaxf(top[1], fmaxf(sc[n][2], sc[n][3]));
+      }
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
+        top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
+      }
+      if (__any_sync(0xffffffffu, top[0] > m[0] || top[1] > m[1])) {  // a row's maximum has grown (multiplying by one else)
+        const float alpha[2] = {exp2f(m[0] - top[0]), exp2f(m[1] - top[1])};
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          m[r] = top[r];
+          l[r] *= alpha[r];
         }
-    }
-    if (kept || base < all_from || base + MMA_KEYS - 1 > all_to) {
-      // (without kept blocks of their own the kept keys lie inside the ordinary blocks: a later row of the tile may see them
-      // although its window starts beyond them; a kept block lies before every row of a tile that has any)
 #pragma unroll
-      for (int n = 0; n < MMA_KEYS / 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int r = e >> 1, key = base + n * 8 + 2 * tig + (e & 1);
-          if (!(kept ? key < keep_first : (key <= pos[r] && (key >= low[r] || (kept_blocks == 0 && key < keep_first))))) sc[n][e] = -INFINITY;
+        for (int i = 0; i < V / 8; ++i) {
+          o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
+          o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
         }
-    }
-    float top[2] = {-FLT_MAX, -FLT_MAX};
+      }
 #pragma unroll
-    for (int n = 0; n < MMA_KEYS / 8; ++n) {
-      top[0] = fmaxf(top[0], fmaxf(sc[n][0], sc[n][1]));
-      top[1] = fmaxf(top[1], fmaxf(sc[n][2], sc[n][3]));
-    }
-    float alpha[2];
+      for (int kk = 0; kk < MMA_PART / 16; ++kk) {
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
-      top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
-      const float m_new = fmaxf(m[r], top[r]);
-      alpha[r] = exp2f(m[r] - m_new);
-      m[r] = m_new;
-      l[r] *= alpha[r];
-    }
+        for (int n = 2 * kk; n < 2 * kk + 2; ++n)
 #pragma unroll
-    for (int i = 0; i < V / 8; ++i) {
-      o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
-      o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
-    }
+          for (int e = 0; e < 4; ++e) {
+            sc[n][e] = exp2f(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
+            l[e >> 1] += sc[n][e];
+          }
+        uint32_t hi[4], lo[4];
+        split_bf16(sc[2 * kk][0], sc[2 * kk][1], hi[0], lo[0]);
+        split_bf16(sc[2 * kk][2], sc[2 * kk][3], hi[1], lo[1]);
+        split_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1], hi[2], lo[2]);
+        split_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3], hi[3], lo[3]);
 #pragma unroll
-    for (int kk = 0; kk < MMA_KEYS / 16; ++kk) {
-#pragma unroll
-      for (int n = 2 * kk; n < 2 * kk + 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          sc[n][e] = exp2f(sc[n][e] - m[e >> 1]);  // a masked score is -inf: weight 0
-          l[e >> 1] += sc[n][e];
+        for (int nv = 0; nv < V / 8; nv += 2) {
+          if (nv * 8 >= vdim) break;
+          uint32_t b[4];  // (values in an odd number of eights: the last columns read 16 bytes beyond the row, and nobody stores them)
+          rows_ldmatrix4_trans(b, src + (uint32_t)((kk * 16 + (lmat & 1) * 8 + lrow) * pitch + dim + nv * 8 + (lmat >> 1) * 8) * 2);
+          mma_16816(o[nv], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+          mma_16816(o[nv + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+          mma_16816(o[nv], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+          mma_16816(o[nv + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
         }
-      uint32_t hi[4], lo[4];
-      split_bf16(sc[2 * kk][0], sc[2 * kk][1], hi[0], lo[0]);
-      split_bf16(sc[2 * kk][2], sc[2 * kk][3], hi[1], lo[1]);
-      split_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1], hi[2], lo[2]);
-      split_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3], hi[3], lo[3]);
-#pragma unroll
-      for (int nv = 0; nv < V / 8; nv += 2) {
-        if (nv * 8 >= vdim) break;
-        uint32_t b[4];  // (values in an odd number of eights: the last columns read 16 bytes beyond the row, and nobody stores them)
-        rows_ldmatrix4_trans(b, src + (uint32_t)((kk * 16 + (lmat & 1) * 8 + lrow) * pitch + dim + nv * 8 + (lmat >> 1) * 8) * 2);
-        mma_16816(o[nv], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
-        mma_16816(o[nv + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
-        mma_16816(o[nv], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
-        mma_16816(o[nv + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
       }
     }
   }
@@ -1072,7 +1092,8 @@ PSB_API int psb_attention_biased_mma(const void* q, const void* kv, const void* 
   if (items < 1 || T < 1 || min_tokens < 1) return 0;
   // two heads that read the same keys and values share a block (64 tokens each) where there are such heads
   const int heads_here = (hq / hkv) % 2 == 0 ? 2 : 1, tile_tokens = 16 * MMA_WARPS / heads_here;
-  const dim3 grid(hq / heads_here, (T + tile_tokens - 1) / tile_tokens + items);
+  const int by_chunk = items == 1 && chunk >= 2 * tile_tokens ? chunk / tile_tokens : 0;  // tiles of a last chunk that is cut off
+  const dim3 grid(hq / heads_here, (T + tile_tokens - 1) / tile_tokens + items + by_chunk);
   if (grid.y > 65535) PSB_REFUSE("attention_biased_mma: %d tokens are too many for one launch", T);
   const size_t smem = mma_smem(dim, vdim, bias != nullptr, heads_here);
 #define MMA_CASE(D_, V_)                                                                                                       \
