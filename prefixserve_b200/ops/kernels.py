@@ -977,7 +977,7 @@ def attention_over_rows(q: torch.Tensor, kv: torch.Tensor, table: torch.Tensor, 
         if (both16 and ROWS_SINGLE and kv.data_ptr() % 16 == 0 and q.data_ptr() % 4 == 0
                 and bool(lib().psb_attention_rows_single_supported(num_heads, num_kv_heads, dim, vdim))):
             blocks = t * num_kv_heads * -(-(num_heads // num_kv_heads) // 16)
-            splits = max(1, min(16, -(-ROWS_BLOCKS_WANTED // max(blocks, 1)), keys // 64))
+            splits = max(1, min(16, -(-ROWS_BLOCKS_WANTED // max(blocks, 1)), keys // 128))
             partial = torch.empty((t, num_heads, splits, vdim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
             check(lib().psb_attention_rows_single(q.data_ptr(), kv.data_ptr(), table.data_ptr(), table.shape[1], positions.data_ptr(),
                                                   token_item.data_ptr(), _ptr(bias), _ptr(sink), out.data_ptr(), t, num_heads, num_kv_heads,
