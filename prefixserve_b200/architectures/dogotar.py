@@ -92,9 +92,13 @@ def dogotar_tensor_name(path: str) -> str:
 
 
 def _without_reader(cfg: DogotarConfig, name: str) -> bool:
-    """The norm in front of a feed-forward that a layer does not have, should a checkpoint carry one."""
-    m = re.match(r"^l(\d+)\.norm2(\.b)?$", name)
-    return bool(m) and int(m.group(1)) < len(cfg.layers) and cfg.layers[int(m.group(1))].ff is None
+    """What a checkpoint may carry although its layer has no use for it: the norm in front of a feed-forward that is not there,
+    the share of a layer that does not mix values."""
+    m = re.match(r"^l(\d+)\.(norm2|norm2\.b|mix\.vmix)$", name)
+    if not m or int(m.group(1)) >= len(cfg.layers):
+        return False
+    layer = cfg.layers[int(m.group(1))]
+    return not getattr(layer.mixer, "v_mix", False) if m.group(2) == "mix.vmix" else layer.ff is None
 
 
 DOGOTAR = Architecture(

@@ -192,9 +192,9 @@ class DogotarConfig:
             layers=tuple(layers),
             stop_token_ids=frozenset(stops),
         )
-        sizes = {(layer.mixer.kv_heads, layer.mixer.vdim) for layer in layers if getattr(layer.mixer, "v_mix", False)}
+        sizes = {layer.mixer.kv_heads * layer.mixer.vdim for layer in layers if getattr(layer.mixer, "v_mix", False)}
         if len(sizes) > 1:
-            raise UnsupportedModelError(f"config.json: layers that mix values must agree in value heads and their size, not {sorted(sizes)}")
+            raise UnsupportedModelError(f"config.json: layers that mix values must have as many value channels, not {sorted(sizes)}")
         return cfg
 
     def to_config_json(self) -> dict[str, Any]:

@@ -65,7 +65,7 @@ CONFIGS = {
         attention(4, 1, 16, 9, 0.3, None, None, (16, 5000.0, None), v_mix=True, mlp=None),
         parallel(left(2, 2, 6, 14, 0.4, None, None), right(1, 9, 20, 12.0), (-0.5, 2.0), None),
         attention(2, 1, 10, 9, 0.33, 9.0, 33, None, v_mix=True, mlp=dense(17)),
-        attention(3, 1, 8, 9, 0.5, 3.0, 14, (2, 40.0, 5.0), v_mix=True, mlp=dense(24)),
+        attention(9, 3, 8, 3, 0.5, 3.0, 14, (2, 40.0, 5.0), v_mix=True, mlp=dense(24)),
     ], vocab=131, width=40, eps=4e-3),
     # sizes in the multiples the tensor-core kernels and the wide accesses take, gaps and none between joined rows
     "wide": config([

@@ -88,7 +88,7 @@ def attention(h, m, w, name, eps, mask, rot=None, v_mix=False, first=None):
     if rot is not None:
         turn = (int(rot["dims"]), float(rot["base"]), float((rot.get("scaling") or {}).get("factor", 1.0)))
         q, k = rotate(q, *turn), rotate(k, *turn)
-    v = mix_values(own, first, weight(w, f"{name}.vmix")) if v_mix and first is not None else own
+    v = mix_values(own, first.view_as(own), weight(w, f"{name}.vmix")) if v_mix and first is not None else own
     k, v = k.repeat_interleave(H // G, dim=1), v.repeat_interleave(H // G, dim=1)
     return capped_attention(q, k, v, float(m["scale"]), m.get("softcap"), mask).reshape(h.shape[0], -1), own
 

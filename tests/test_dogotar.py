@@ -77,12 +77,13 @@ def test_every_tensor_of_a_checkpoint_has_a_part_and_the_cache_holds_what_the_ma
                 assert (need.paged.window, need.paged.chunk) == (None, size) and held <= need.state.shape[0] <= held + 3
 
 
-def test_a_norm_without_a_feed_forward_may_be_left_in_a_checkpoint_but_nothing_else(tmp_path):
+def test_what_a_layer_has_no_use_for_may_be_left_in_a_checkpoint_but_nothing_else(tmp_path):
     from prefixserve_b200 import architectures  # noqa: F401
     from prefixserve_b200.config.registry import get_architecture, read_model_folder
     arch, typed = read_model_folder(dm.write_folder(tmp_path / "m", dm.CONFIGS["mixed"], {}))
     assert arch is get_architecture("Dogotar")
-    assert arch.ignorable(typed, "l2.norm2") and arch.ignorable(typed, "l3.norm2.b")
+    assert arch.ignorable(typed, "l2.norm2") and arch.ignorable(typed, "l3.norm2.b") and arch.ignorable(typed, "l0.mix.vmix")
+    assert not arch.ignorable(typed, "l4.mix.vmix")
     assert not arch.ignorable(typed, "l0.norm2") and not arch.ignorable(typed, "l2.norm1") and not arch.ignorable(typed, "l9.norm2")
 
 
